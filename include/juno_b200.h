@@ -48,6 +48,7 @@ typedef struct juno_model juno_model;
 typedef struct juno_seq juno_seq;
 typedef struct juno_kvpool juno_kvpool;
 typedef struct juno_gguf juno_gguf;
+typedef struct juno_safetensors juno_safetensors;
 
 /* Thread-local text of the last failure on the calling thread. */
 const char *juno_last_error(void);
@@ -214,6 +215,22 @@ int juno_gguf_tensor(juno_gguf *g, const char *name, int32_t *ggml_type, int32_t
                      const void **data, int64_t *n_bytes);
 int juno_gguf_raw_byte_count(int32_t ggml_type, int64_t n_elems, int64_t *bytes); /* rawByteCount :347-360 */
 
+/* ── safetensors files (host only, no GPU needed) ──────────────────────────────
+ * The container of a model folder: 8-byte little-endian header length, a JSON object name -> dtype, shape, data_offsets,
+ * then the data.  Mapped read-only; tensor pointers stay valid until juno_safetensors_close.  A damaged file gives
+ * JUNO_ERR_INVALID_ARG. */
+#define JUNO_ST_BF16 0
+#define JUNO_ST_F16 1
+#define JUNO_ST_F32 2
+#define JUNO_ST_I32 3 /* any other element type reads as -1 */
+int juno_safetensors_open(const char *path, juno_safetensors **out);
+int juno_safetensors_close(juno_safetensors *s);
+int juno_safetensors_count(juno_safetensors *s, int64_t *n_tensors);
+int juno_safetensors_name(juno_safetensors *s, int64_t index, char *buf, int32_t buf_len); /* in order of the data */
+/* dims8 is outermost first, unused entries 1; n_dims 0 = a single number.  Any output pointer may be null. */
+int juno_safetensors_tensor(juno_safetensors *s, const char *name, int32_t *dtype, int32_t *n_dims, int64_t *dims8,
+                            const void **data, int64_t *n_bytes);
+
 /* Host-only (no GPU needed): the slice of a FULL tensor of `kind` that rank tp_rank of tp_world keeps - the rule
  * juno_model_set_tensor applies itself (TensorShardContext.java:74-100: headsPerNode = numHeads / world, sliceDim =
  * hidden / world).  out6 = {rows, cols, row0, nrows, col0, ncols} of the full tensor and of the kept sub-matrix:
@@ -243,6 +260,34 @@ int juno_gguf_model_cfg(juno_gguf *g, juno_model_cfg *cfg);
  * juno_model_set_tensor, straight from the mapped file; attn_{q,k,v}.bias of every layer too when blk.0.attn_q.bias exists.
  * Call juno_model_finalize afterwards. */
 int juno_model_load_gguf(juno_model *m, juno_gguf *g);
+/* ── model registry ────────────────────────────────────────────────────────────
+ * Opens a model by what the path holds and returns it finalized, ready for juno_model_seq_create and the step calls:
+ *   - a folder with config.json and model.safetensors: the design that config.json's "architecture" names.  Registered:
+ *     "Vosotar" (latent attention without positions over latent pages, squared-ReLU feed-forwards, scalar norms, a short
+ *     convolution on the mixer's input whose state belongs to the sequence, sigmoid-gated residuals).  An architecture
+ *     that is not registered gives JUNO_ERR_UNSUPPORTED;
+ *   - a file: GGUF, the quantised LLaMA family (juno_gguf_model_cfg, juno_model_load_gguf).
+ * Sequences of a model with a convolution state can be continued at their end, restarted at 0, or rewound by the few
+ * positions the state reaches back; anything else is JUNO_ERR_INVALID_ARG.  One GPU. */
+#define JUNO_DTYPE_DEFAULT 0 /* folder: BF16 products and pages with FP32 norms, scores, sums and state; GGUF: FP16 pages */
+#define JUNO_DTYPE_F32 1     /* folder: everything in true 32-bit; GGUF: FP32 pages */
+typedef struct juno_open_opts {
+    int32_t struct_size; /* sizeof(juno_open_opts) */
+    int32_t max_batch;   /* most sequences per step */
+    int32_t max_seqs;    /* most live sequences */
+    int32_t max_ctx;     /* most positions per sequence */
+    int32_t dtype;       /* JUNO_DTYPE_* */
+    int32_t max_rows;    /* most prompt positions per pass of juno_prefill (0 = 2048); GGUF models: 64 at most */
+} juno_open_opts;
+int juno_model_open(juno_ctx *ctx, const char *path, const juno_open_opts *opts, juno_model **out);
+typedef struct juno_model_info {
+    char architecture[32];
+    int32_t hidden, n_layers, vocab, max_batch, max_seqs, max_ctx, max_rows, reserved;
+    int64_t weight_bytes;          /* bytes of weights a one-token step reads (0: not kept for this family) */
+    int64_t cache_bytes_per_token; /* all layers */
+    int64_t state_bytes_per_seq;   /* convolution state, all layers */
+} juno_model_info;
+int juno_model_describe(juno_model *m, juno_model_info *info);
 int juno_model_free(juno_model *m); /* releaseGpuResources (LlamaTransformerHandler.java:424-448) */
 /* How a finalized model exchanges the partial products of its row-parallel projections: 0 = one GPU (nothing to
  * exchange), 1 = NCCL all-reduce, 2 = stores into peer-mapped inboxes by the producing kernels (up to eight
@@ -263,6 +308,11 @@ int juno_forward(juno_model *m, int32_t n, juno_seq *const *seqs, const int32_t 
  * optional and refer to the LAST position fed.  Tensor parallel models: logits only with an unsharded vocabulary. */
 int juno_prefill(juno_model *m, juno_seq *seq, const int32_t *token_ids, int32_t n_tokens, int32_t start_pos,
                  float *logits_host, int32_t *argmax_out);
+
+/* The same passes with logits at chosen places of the portion: want[i] in [0, n_tokens), logits_host [n_want][vocab] in
+ * that order (n_want may be 0). */
+int juno_prefill_logits(juno_model *m, juno_seq *seq, const int32_t *token_ids, int32_t n_tokens, int32_t start_pos,
+                        int32_t n_want, const int32_t *want, float *logits_host);
 
 /* `steps` greedy steps kept on the device: step 0 feeds first_tokens at positions, step s>0
  * feeds the token picked at step s-1 at positions+s.  out_ids is [steps][n]. */
@@ -287,8 +337,9 @@ int juno_ctx_counters(juno_ctx *ctx, juno_counters *out, int32_t reset);
  * without CUDA graphs; juno_ctx_profile_read synchronises and returns, per category, launches, summed
  * milliseconds and the algorithmic bytes the launches had to move.  Categories: 0 Q4_K GEMV, 1 Q6_K GEMV,
  * 2 Q8_0 GEMV, 3 attention (split + merge), 4 RoPE + KV append, 5 other, 6 batched products that ran on the
- * tcgen05/TMEM kernel (also counted under their block format). */
-#define JUNO_PROF_COUNT 7
+ * tcgen05/TMEM kernel (also counted under their block format); layer stacks with dense weights: 7 matrix products of many
+ * rows, 8 fused products of a decode step, 9 row-wise operations (their attention counts under 3). */
+#define JUNO_PROF_COUNT 10
 typedef struct juno_profile_entry {
     int64_t launches;
     double ms;

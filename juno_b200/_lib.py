@@ -24,6 +24,16 @@ class ModelCfg(C.Structure):
                 ("kv_dtype", C.c_int32), ("tp_rank", C.c_int32), ("tp_world", C.c_int32), ("nccl_id", C.c_uint8 * 128)]
 
 
+class OpenOpts(C.Structure):
+    _fields_ = [(k, C.c_int32) for k in ("struct_size", "max_batch", "max_seqs", "max_ctx", "dtype", "max_rows")]
+
+
+class ModelInfo(C.Structure):
+    _fields_ = [("architecture", C.c_char * 32)] + [(k, C.c_int32) for k in ("hidden", "n_layers", "vocab", "max_batch", "max_seqs",
+                "max_ctx", "max_rows", "reserved")] + [(k, C.c_int64) for k in ("weight_bytes", "cache_bytes_per_token",
+                "state_bytes_per_seq")]
+
+
 class Counters(C.Structure):
     _fields_ = [("kernel_launches", C.c_int64), ("gemv_calls", C.c_int64), ("forward_calls", C.c_int64),
                 ("h2d_bytes", C.c_int64), ("d2h_bytes", C.c_int64)]
@@ -33,7 +43,7 @@ class ProfileEntry(C.Structure):
     _fields_ = [("launches", C.c_int64), ("ms", C.c_double), ("algo_bytes", C.c_double)]
 
 
-PROF_NAMES = ["gemv_q4k", "gemv_q6k", "gemv_q8_0", "attention", "rope_append", "other", "gemm_tcgen05"]
+PROF_NAMES = ["gemv_q4k", "gemv_q6k", "gemv_q8_0", "attention", "rope_append", "other", "gemm_tcgen05", "gemm_rows", "gemv_rows", "row_ops"]
 
 P = C.c_void_p
 PP = C.POINTER(C.c_void_p)
@@ -94,6 +104,14 @@ SIGNATURES = {
     "juno_gguf_raw_byte_count": (C.c_int, [I32, I64, C.POINTER(I64)]),
     "juno_gguf_model_cfg": (C.c_int, [P, C.POINTER(ModelCfg)]),
     "juno_model_load_gguf": (C.c_int, [P, P]),
+    "juno_safetensors_open": (C.c_int, [C.c_char_p, PP]),
+    "juno_safetensors_close": (C.c_int, [P]),
+    "juno_safetensors_count": (C.c_int, [P, C.POINTER(I64)]),
+    "juno_safetensors_name": (C.c_int, [P, I64, C.c_char_p, I32]),
+    "juno_safetensors_tensor": (C.c_int, [P, C.c_char_p, C.POINTER(I32), C.POINTER(I32), C.POINTER(I64), PP, C.POINTER(I64)]),
+    "juno_model_open": (C.c_int, [P, C.c_char_p, C.POINTER(OpenOpts), PP]),
+    "juno_model_describe": (C.c_int, [P, C.POINTER(ModelInfo)]),
+    "juno_prefill_logits": (C.c_int, [P, P, P, I32, I32, I32, P, P]),
 }
 
 _lib = None

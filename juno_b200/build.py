@@ -16,7 +16,8 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libjuno_b200.so")
-SOURCES = ["context.cu", "gemv.cu", "qgemv.cu", "gemm.cu", "gemm_tc.cu", "attn.cu", "model.cu", "gguf_file.cu"]
+SOURCES = ["context.cu", "gemv.cu", "qgemv.cu", "gemm.cu", "gemm_tc.cu", "attn.cu", "model.cu", "gguf_file.cu",
+           "safetensors_file.cu", "registry.cu", "vosotar.cu", "stack.cu", "rowops.cu", "gemm_rows.cu", "latent_attn.cu"]
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 
 
@@ -31,7 +32,7 @@ def _newest_header() -> float:
     t = 0.0
     for root in (CSRC, os.path.join(HERE, "..", "include")):
         for f in os.listdir(root):
-            if f.endswith((".cuh", ".h")):
+            if f.endswith((".cuh", ".h", ".hpp")):
                 t = max(t, os.path.getmtime(os.path.join(root, f)))
     return t
 
@@ -51,9 +52,12 @@ def _compile(src: str, verbose: bool) -> str:
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
-    os.makedirs(OBJ, exist_ok=True)
     srcs = [s for s in SOURCES if os.path.exists(os.path.join(CSRC, s))]
     hdr_t = _newest_header()
+    newest = max([hdr_t] + [os.path.getmtime(os.path.join(CSRC, s)) for s in srcs])
+    if not force and os.path.exists(LIB) and os.path.getmtime(LIB) > newest:
+        return LIB
+    os.makedirs(OBJ, exist_ok=True)
     todo = []
     for s in srcs:
         obj = os.path.join(OBJ, s.replace(".cu", ".o"))

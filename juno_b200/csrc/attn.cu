@@ -937,6 +937,72 @@ int kvpool_create(juno_ctx *ctx, int n_layers, int n_kv_heads, int head_dim, int
     return JUNO_OK;
 }
 
+int kvpool_create_latent(juno_ctx *ctx, const std::vector<int> &row_width, int n_pages, int dtype, int max_slots, int max_pages_per_seq,
+                         int state_ring, int state_width, int state_taps, juno_kvpool **out) {
+    JUNO_REQUIRE(!row_width.empty() && n_pages > 0 && max_slots > 0 && max_pages_per_seq > 0, "bad latent pool geometry");
+    JUNO_REQUIRE(dtype == 1 || dtype == 2, "latent rows are FP32 (1) or BF16 (2), not %d", dtype);
+    JUNO_REQUIRE(state_ring >= 0 && (state_ring & (state_ring - 1)) == 0 && (state_ring == 0 || state_ring >= 2 * state_taps),
+                 "a state of %d positions does not fit a convolution of %d taps", state_ring, state_taps);
+    juno_kvpool *p = new juno_kvpool();
+    p->magic = kMagicPool;
+    p->ctx = ctx;
+    p->latent = true;
+    p->n_layers = (int)row_width.size();
+    p->n_kv_heads = 1;
+    p->head_dim = *std::max_element(row_width.begin(), row_width.end());
+    p->n_pages = n_pages;
+    p->dtype = dtype;
+    p->page_tokens = kPageTokens;
+    p->elem_bytes = dtype == 2 ? 2 : 4;
+    p->max_slots = max_slots;
+    p->max_pages_per_seq = max_pages_per_seq;
+    p->k = p->v = nullptr;
+    p->d_table = p->h_table = nullptr;
+    p->owned_by_model = 0;
+    p->row_width = row_width;
+    size_t elems = 0;
+    for (int w : row_width) {
+        p->row_off.push_back(elems);
+        elems += (size_t)n_pages * kPageTokens * w;
+    }
+    p->state_ring = state_ring;
+    p->state_width = state_width;
+    p->state_taps = state_taps;
+    const size_t bytes = elems * p->elem_bytes, tbytes = (size_t)max_slots * max_pages_per_seq * sizeof(int32_t);
+    const size_t sbytes = (size_t)max_slots * p->n_layers * state_ring * state_width * sizeof(float);
+    cudaError_t e = cudaMalloc(&p->k, bytes);
+    if (e == cudaSuccess && sbytes) e = cudaMalloc((void **)&p->state, sbytes);
+    if (e == cudaSuccess) e = cudaMalloc((void **)&p->d_table, tbytes);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&p->h_table, tbytes);
+    if (e == cudaSuccess) e = cudaMemsetAsync(p->d_table, 0, tbytes, ctx->stream);
+    if (e == cudaSuccess) e = cudaMemsetAsync(p->k, 0, bytes, ctx->stream);
+    if (e == cudaSuccess && sbytes) e = cudaMemsetAsync(p->state, 0, sbytes, ctx->stream);
+    if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        set_error("cudaMalloc of the latent pool (%zu + %zu bytes) failed: %s", bytes, sbytes, cudaGetErrorString(e));
+        if (p->k) cudaFree(p->k);
+        if (p->state) cudaFree(p->state);
+        if (p->d_table) cudaFree(p->d_table);
+        if (p->h_table) cudaFreeHost(p->h_table);
+        delete p;
+        return e == cudaErrorMemoryAllocation ? JUNO_ERR_OOM : JUNO_ERR_CUDA;
+    }
+    memset(p->h_table, 0, tbytes);
+    for (int i = n_pages - 1; i >= 0; i--) p->free_pages.push_back(i);
+    p->page_refs.assign((size_t)n_pages, 0);
+    for (int i = max_slots - 1; i >= 0; i--) p->free_slots.push_back(i);
+    *out = p;
+    return JUNO_OK;
+}
+
+int seq_resume_check(const juno_kvpool *p, int len, int pos) {
+    if (p->state_ring == 0 || pos <= 0 || std::max(0, pos - (p->state_taps - 1)) >= len - p->state_ring) return JUNO_OK;
+    set_error("position %d: the layer state of this sequence reaches back to position %d only (%d cached positions); start over at 0",
+              pos, len - p->state_ring + p->state_taps - 1, len);
+    return JUNO_ERR_INVALID_ARG;
+}
+
 int kvpool_destroy(juno_kvpool *p) {
     if (!p) return JUNO_ERR_INVALID_ARG;
     if (p->magic != kMagicPool) {
@@ -947,8 +1013,10 @@ int kvpool_destroy(juno_kvpool *p) {
     cudaStreamSynchronize(p->ctx->stream);
     cudaFree(p->k);
     cudaFree(p->v);
+    if (p->state) cudaFree(p->state);
     cudaFree(p->d_table);
     cudaFreeHost(p->h_table);
+    p->state = nullptr;
     p->k = p->v = nullptr;
     p->magic = kMagicDead;
     return JUNO_OK;
@@ -976,6 +1044,14 @@ int seq_create(juno_kvpool *p, int max_tokens, juno_seq **out) {
 
 // Copies one page (all layers, K and V) to another on the device, ordered on `st`.
 static int page_copy(juno_kvpool *p, int dst, int src, cudaStream_t st) {
+    if (p->latent) {
+        for (int layer = 0; layer < p->n_layers; layer++) {
+            const size_t page_bytes = (size_t)kPageTokens * p->row_width[layer] * p->elem_bytes;
+            uint8_t *plane = static_cast<uint8_t *>(p->k) + p->row_off[layer] * p->elem_bytes;
+            JUNO_CUDA_TRY(cudaMemcpyAsync(plane + dst * page_bytes, plane + src * page_bytes, page_bytes, cudaMemcpyDeviceToDevice, st));
+        }
+        return JUNO_OK;
+    }
     const size_t page_bytes = (size_t)p->n_kv_heads * kPageTokens * p->head_dim * p->elem_bytes;
     for (int layer = 0; layer < p->n_layers; layer++) {
         const size_t d = ((size_t)layer * p->n_pages + dst) * page_bytes, s = ((size_t)layer * p->n_pages + src) * page_bytes;
@@ -1103,8 +1179,20 @@ int juno_seq_fork(juno_seq *src, int32_t n_tokens, juno_seq **out) {
     juno_kvpool *p = src->pool;
     std::lock_guard<std::recursive_mutex> lk(p->ctx->mu);
     DeviceGuard g(p->ctx->device);
+    JUNO_TRY(seq_resume_check(p, src->len, n_tokens));
     juno_seq *s = nullptr;
     JUNO_TRY(seq_create(p, src->max_tokens, &s));
+    if (p->state) {  // the state is small and changes every step: each holder has its own
+        const size_t slot_floats = (size_t)p->n_layers * p->state_ring * p->state_width;
+        const cudaError_t e = cudaMemcpyAsync(p->state + s->slot * slot_floats, p->state + src->slot * slot_floats, slot_floats * sizeof(float),
+                                              cudaMemcpyDeviceToDevice, p->ctx->stream);
+        if (e != cudaSuccess) {
+            p->free_slots.push_back(s->slot);
+            s->magic = kMagicDead;
+            delete s;
+            JUNO_CUDA_TRY(e);
+        }
+    }
     const int n_pg = (n_tokens + kPageTokens - 1) / kPageTokens;
     int32_t *row = p->h_table + (size_t)s->slot * p->max_pages_per_seq;
     for (int i = 0; i < n_pg; i++) {
@@ -1142,6 +1230,7 @@ int juno_seq_append_kv(juno_seq *s, int32_t layer, int32_t pos, int32_t n_tokens
     juno_kvpool *p = s->pool;
     juno_ctx *c = p->ctx;
     JUNO_REQUIRE(k_host && v_host, "null K/V");
+    JUNO_REQUIRE(!p->latent, "this sequence belongs to a model with latent pages: it has no K and V to append");
     JUNO_REQUIRE(layer >= 0 && layer < p->n_layers, "layer %d out of range", layer);
     JUNO_REQUIRE(pos >= 0 && n_tokens >= 0, "bad position range");
     if (n_tokens == 0) return JUNO_OK;

@@ -5,10 +5,21 @@
 #include "common.cuh"
 
 // Page layout (both K and V): [layer][page][kv_head][page_tokens=16][head_dim], FP16 or FP32.
+//
+// A LATENT pool keeps one row per position and layer instead (attention whose keys and values are linear in a small latent):
+// only `k` exists, layer l is the plane [page][page_tokens][row_width[l]] that starts at element row_off[l], BF16 or FP32.
+// Beside the pages it can hold a position-addressed state for every slot: [slot][layer][ring][width] FP32 rows, position p of
+// a sequence at p & (ring - 1), the last `ring` inputs of a short convolution over time.  Zeros before the first position are
+// the readers' business (position < 0), so a slot that is used again needs no clearing.
 struct juno_kvpool {
     uint32_t magic;
     juno_ctx *ctx;
-    int n_layers, n_kv_heads, head_dim, n_pages, dtype;  // dtype 0 = f16, 1 = f32
+    int n_layers, n_kv_heads, head_dim, n_pages, dtype;  // dtype 0 = f16, 1 = f32, 2 = bf16 (latent pools only)
+    bool latent = false;
+    std::vector<int> row_width;
+    std::vector<size_t> row_off;
+    float *state = nullptr;
+    int state_ring = 0, state_width = 0, state_taps = 1;  // a convolution reads state_taps - 1 positions back
     int page_tokens;
     int elem_bytes;
     void *k, *v;
@@ -68,7 +79,13 @@ int launch_rope_append(juno_ctx *ctx, const juno_kvpool *pool, int layer, int n,
 
 int kvpool_create(juno_ctx *ctx, int n_layers, int n_kv_heads, int head_dim, int n_pages, int dtype, int max_slots,
                   int max_pages_per_seq, juno_kvpool **out);
+// Latent pool; row_width[l] elements per position in layer l.  state_ring: a power of two, or 0 for no state.
+int kvpool_create_latent(juno_ctx *ctx, const std::vector<int> &row_width, int n_pages, int dtype, int max_slots, int max_pages_per_seq,
+                         int state_ring, int state_width, int state_taps, juno_kvpool **out);
 int kvpool_destroy(juno_kvpool *p);
+// Can a sequence of this pool that has written `len` positions be continued at `pos`?  Pages allow any pos <= len; the state
+// holds the last state_ring inputs only, so a pool with state can step back by a few positions, or start over at 0.
+int seq_resume_check(const juno_kvpool *p, int len, int pos);
 int seq_create(juno_kvpool *p, int max_tokens, juno_seq **out);
 // Makes sure pages exist for positions [0, upto) and that the device page table row is current (stream-ordered).
 // Makes the positions [from, upto) of the sequence writable: allocates missing pages and gives the sequence a private

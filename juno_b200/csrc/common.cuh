@@ -51,6 +51,8 @@ constexpr uint32_t kMagicSeq = 0x4A534551;    // "JSEQ"
 constexpr uint32_t kMagicPool = 0x4A4B5650;   // "JKVP"
 constexpr uint32_t kMagicDead = 0xDEADDEAD;
 
+constexpr unsigned kErrStackWait = 8;  // code of a given-up wait in a layer stack's kernels (see GemvScratch::qerr)
+
 // Scratch of the host-level MatVec entry points and the word kernels report a given-up wait in.
 struct GemvScratch {
     unsigned *qerr = nullptr;       // device address of qerr_host
@@ -63,7 +65,7 @@ struct GemvScratch {
 }  // namespace juno
 
 namespace juno {
-enum ProfCat { PROF_GEMV_Q4K = 0, PROF_GEMV_Q6K, PROF_GEMV_Q80, PROF_ATTN, PROF_ROPE_APPEND, PROF_OTHER, PROF_GEMM_TC, PROF_COUNT };
+enum ProfCat { PROF_GEMV_Q4K = 0, PROF_GEMV_Q6K, PROF_GEMV_Q80, PROF_ATTN, PROF_ROPE_APPEND, PROF_OTHER, PROF_GEMM_TC, PROF_GEMM_ROWS, PROF_GEMV_ROWS, PROF_ROWOPS, PROF_COUNT };
 struct ProfSpan {
     int cat;
     double bytes;

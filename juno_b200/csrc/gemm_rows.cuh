@@ -1,0 +1,36 @@
+// Matrix products of layer stacks with dense weights: out[m][n] = epilogue(sum_k a[m][k] * w[n][k]), m = positions.
+#pragma once
+#include "rowops.cuh"
+
+namespace juno {
+
+enum GemmEpi {
+    GE_F32 = 0,      // FP32 result
+    GE_OP,           // operand type
+    GE_SIGMOID,      // sigmoid(acc + bias[n]), operand type
+    GE_RELU2,        // max(acc, 0)^2, operand type
+    GE_MUL,          // acc * aux[m][n] (operand type), operand type
+    GE_GROUP_GATE,   // acc * sigmoid(gate[m][group]) (FP32), operand type
+};
+
+// `groups` > 1: a block-diagonal product (one block per attention head): group z multiplies columns a_step*z.. of `a` with rows
+// w_step*z.. of `w` into columns o_step*z.. of `out`; N and K are a group's.
+struct GemmArgs {
+    const void *a = nullptr;
+    int lda = 0;
+    const void *w = nullptr;
+    int ldw = 0;
+    int M = 0, N = 0, K = 0;
+    void *out = nullptr;
+    int ldo = 0;
+    int epi = GE_OP;
+    const float *bias = nullptr;
+    const void *aux = nullptr;
+    int ldaux = 0;
+    int groups = 1, a_step = 0, w_step = 0, o_step = 0;
+    int a_rows = 0;  // rows of `a` that may be read (0: M)
+    int w_rows = 0;  // rows of `w` in memory (0: N, or w_step * groups)
+};
+int launch_gemm_rows(juno_ctx *c, int dt, const GemmArgs &a, unsigned *err, cudaStream_t st);
+
+}  // namespace juno

@@ -18,7 +18,9 @@
 #include "common.cuh"
 #include "dequant.cuh"
 #include "gemv.cuh"
+#include "model.cuh"
 #include "qgemv.cuh"
+#include "stack.cuh"
 
 namespace juno {
 
@@ -28,7 +30,6 @@ namespace juno {
 struct NcclId {
     char internal[128];
 };
-typedef struct ncclComm *NcclComm;
 struct NcclApi {
     void *h = nullptr;
     int (*GetUniqueId)(NcclId *) = nullptr;
@@ -260,72 +261,6 @@ __global__ void ungather_logits_kernel(LogitsView lv, float *out) {
 
 }  // namespace juno
 
-// ───────────────────────────── model object ───────────────────────────────────────────────
-struct JunoLayer {
-    juno_qmat *w[12] = {nullptr};  // indexed by tensor kind (ATTN_Q .. FFN_DOWN); gate and up share w[FFN_GATE]
-    std::vector<uint8_t> gate_host, up_host;  // row slices waiting for their partner
-    int gate_type = -1, up_type = -1;
-    float *attn_norm = nullptr, *ffn_norm = nullptr;
-    float *bqkv = nullptr;  // optional attn_{q,k,v}.bias of this rank, laid out like a row of the q|k|v buffer
-    int bias_seen = 0;      // bit per bias kind received
-};
-
-struct JunoGraph {
-    cudaGraphExec_t exec = nullptr;
-    int launches = 0;
-    int seen = 0;
-};
-
-struct juno_model {
-    uint32_t magic;
-    juno_ctx *ctx;
-    juno_model_cfg cfg;
-    int hd, world, rank;
-    int heads_loc, kv_loc, inter_loc, vocab_loc;  // this rank's share
-    int qkv_ld;
-    bool finalized = false;
-    bool vocab_sharded = false;
-    std::vector<JunoLayer> layers;
-    juno_qmat *tok_embd = nullptr, *output = nullptr;
-    bool output_is_embd = false, output_slice_of_embd = false;
-    float *output_norm = nullptr;
-    juno_kvpool *pool = nullptr;
-    juno::NcclComm comm = nullptr;
-    // activations
-    float *x[2] = {nullptr, nullptr}, *qkv = nullptr, *att = nullptr, *proj = nullptr, *proj2 = nullptr;
-    float *hdn = nullptr, *xsc = nullptr;  // batched path: silu(gate)*up rows; per-row factors of the three FP16 images
-    uint8_t *img_h_tc = nullptr;            // batched path: the hidden-size activation again, chunk-major for the tcgen05 kernel
-    unsigned *tc_err = nullptr;             // device word: a wait inside the tcgen05 kernel gave up
-    bool tc_used = false;                   // the batched path ran since the word was last read
-    uint8_t *img_h = nullptr, *img_att = nullptr, *img_i = nullptr;  // staged activations (K = hidden, local heads, local FFN)
-    float *logits_loc = nullptr, *logits_gather = nullptr, *logits_full = nullptr;
-    float *attn_scratch = nullptr;
-    size_t attn_scratch_floats = 0;
-    float2 *rope_cs = nullptr;
-    int32_t *d_step = nullptr;  // tokens | positions | slots | seq_lens, max_batch each
-    int32_t *d_argmax = nullptr, *d_pidx = nullptr, *d_out_ids = nullptr, *d_step_counter = nullptr;
-    float *d_pval = nullptr;
-    int out_ids_cap = 0;
-    int32_t *h_step = nullptr;  // pinned mirror of d_step
-    int last_n = 0, last_x = 0;
-    double step_kv_bytes = 0;  // K+V bytes one layer's attention reads in the current step
-    std::map<uint64_t, JunoGraph> graphs;
-    bool use_graphs = true, mix_formats = true;  // JUNO_NO_GRAPH / JUNO_NO_MIXED
-    // tensor parallelism without collective calls on the 1..8 sequence path: per-rank exchange buffer (flags + inbox
-    // slots per row-parallel product), mapped into every peer (CUDA IPC), see enqueue_layers_q
-    bool tp_push = false;
-    uint8_t *tp_buf = nullptr;           // this rank's buffer
-    uint8_t *tp_peer[8] = {nullptr};     // every rank's buffer as seen from here (tp_peer[rank] == tp_buf)
-    size_t tp_inbox_off = 0, tp_pair_off = 0;
-    int tp_bq = 0;                       // sequences an inbox slot holds
-    unsigned *tp_failed = nullptr;       // device word: a wait for another rank ran out during this step
-    float *tp_red = nullptr;             // [2 * n_layers][tp_bq][hidden] (value, step) pairs: the ranks' partials added by the first CTAs
-    bool tp_reduce = false;              // consumers poll tp_red instead of every rank's inbox (four ranks and more)
-    bool comm_failed = false;            // a collective timed out or NCCL reported an asynchronous error: no further steps
-    unsigned *tp_epoch = nullptr;        // step number, incremented on the device at the start of every step
-    int batched_from = 9;  // smallest batch on the FP16 one-pass kernels (JUNO_GEMM_MIN_BATCH, read when the model is created)
-};
-
 namespace juno {
 
 static int model_check(juno_model *m) {
@@ -412,6 +347,8 @@ static void model_release(juno_model *m) {
     for (void *b : bufs)
         if (b) cudaFree(b);
     if (m->h_step) cudaFreeHost(m->h_step);
+    stack_free(m->stack);
+    m->stack = nullptr;
     m->magic = kMagicDead;
 }
 
@@ -588,6 +525,8 @@ int juno_model_create(juno_ctx *c, const juno_model_cfg *cfg, juno_model **out) 
     m->vocab_sharded = (w > 1) && (cfg->vocab % w == 0);
     m->vocab_loc = m->vocab_sharded ? cfg->vocab / w : cfg->vocab;
     m->qkv_ld = (m->heads_loc + 2 * m->kv_loc) * hd;
+    m->step_cap = cfg->max_batch;
+    m->logit_cap = cfg->max_batch;
     m->layers.resize(cfg->n_layers);
     const char *ng = getenv("JUNO_NO_GRAPH");
     m->use_graphs = !(ng && *ng == '1');
@@ -622,6 +561,7 @@ int juno_model_set_tensor(juno_model *m, int32_t kind, int32_t layer, const void
                           int64_t cols) {
     JUNO_TRY(model_check(m));
     JUNO_REQUIRE(blocks, "blocks is null");
+    JUNO_REQUIRE(!m->stack, "a model opened from a folder has loaded its tensors already");
     JUNO_REQUIRE(!m->finalized, "model is already finalized");
     JUNO_REQUIRE(kind >= 0 && kind <= JUNO_T_ATTN_V_BIAS, "unknown tensor kind %d", kind);
     juno_ctx *c = m->ctx;
@@ -703,6 +643,74 @@ int juno_model_set_tensor(juno_model *m, int32_t kind, int32_t layer, const void
 }  // extern "C"
 
 // ───────────────────────────── finalize ───────────────────────────────────────────────────
+namespace juno {
+// What every model family's step uses: tokens, positions, slots and lengths of its rows, and the greedy pick.
+static int alloc_step_buffers(juno_model *m) {
+    const int B = m->cfg.max_batch, S = m->step_cap;
+    JUNO_TRY(dev_alloc((void **)&m->d_step, (size_t)4 * S * 4));
+    JUNO_TRY(dev_alloc((void **)&m->d_argmax, (size_t)B * 4));
+    JUNO_TRY(dev_alloc((void **)&m->d_pidx, (size_t)B * kArgmaxBlocks * 4));
+    JUNO_TRY(dev_alloc((void **)&m->d_pval, (size_t)B * kArgmaxBlocks * 4));
+    JUNO_TRY(dev_alloc((void **)&m->d_step_counter, 4));
+    JUNO_CUDA_TRY(cudaMallocHost((void **)&m->h_step, (size_t)4 * S * 4));
+    return JUNO_OK;
+}
+
+constexpr int kStackDefaultRows = 2048;  // positions per pass of a prompt, when the caller does not say
+constexpr int kStackLogitRows = 64;      // logits computed at once inside a prompt
+
+int model_from_stack(juno_ctx *c, StackNet *net, const char *architecture, const juno_open_opts &o, juno_model **out) {
+    const StackSpec &s = net->spec;
+    juno_model *m = new juno_model();
+    m->magic = kMagicModel;
+    m->ctx = c;
+    m->stack = net;
+    m->architecture = architecture;
+    memset(&m->cfg, 0, sizeof(m->cfg));
+    m->cfg.struct_size = (int32_t)sizeof(m->cfg);
+    m->cfg.hidden = s.width;
+    m->cfg.n_layers = (int32_t)s.layers.size();
+    m->cfg.vocab = s.vocab;
+    m->cfg.rms_eps = s.eps;
+    m->cfg.max_batch = o.max_batch;
+    m->cfg.max_seqs = o.max_seqs;
+    m->cfg.max_ctx = o.max_ctx;
+    m->cfg.tp_world = 1;
+    m->world = 1;
+    m->rank = 0;
+    m->vocab_loc = s.vocab;
+    m->step_cap = std::max(o.max_batch, std::min(o.max_rows > 0 ? o.max_rows : kStackDefaultRows, o.max_ctx));
+    m->logit_cap = std::max(o.max_batch, std::min(kStackLogitRows, m->step_cap));
+    const char *ng = getenv("JUNO_NO_GRAPH");
+    m->use_graphs = !(ng && *ng == '1');
+    auto build = [&]() -> int {
+        std::vector<int> widths;
+        for (const StackLayerSpec &L : s.layers) widths.push_back(L.mix.rp());
+        const int pages_per_seq = (o.max_ctx + kPageTokens - 1) / kPageTokens;
+        const long long pages = (long long)o.max_seqs * pages_per_seq;
+        JUNO_REQUIRE(pages < (1ll << 31), "latent pool too large");
+        int ring = 0;
+        if (s.taps > 1)
+            for (ring = 16; ring < 2 * s.taps; ring <<= 1) {
+            }
+        JUNO_TRY(kvpool_create_latent(c, widths, (int)pages, net->dt == DT_F32 ? 1 : 2, o.max_seqs, pages_per_seq, ring, s.wp(), s.taps, &m->pool));
+        m->pool->owned_by_model = 1;
+        JUNO_TRY(stack_alloc(c, net, o.max_batch, m->step_cap, m->logit_cap));
+        JUNO_TRY(dev_alloc((void **)&m->logits_loc, (size_t)m->logit_cap * s.vocab * 4));
+        return alloc_step_buffers(m);
+    };
+    const int rc = build();
+    if (rc != JUNO_OK) {
+        model_release(m);
+        delete m;
+        return rc;
+    }
+    m->finalized = true;
+    *out = m;
+    return JUNO_OK;
+}
+}  // namespace juno
+
 extern "C" int juno_model_finalize(juno_model *m) {
     JUNO_TRY(model_check(m));
     if (m->finalized) return JUNO_OK;
@@ -754,12 +762,7 @@ extern "C" int juno_model_finalize(juno_model *m) {
     m->attn_scratch_floats = (size_t)(c->sm_count * 4 + B * m->kv_loc) * (m->heads_loc / m->kv_loc) * (hd + 2) + 64;
     JUNO_TRY(dev_alloc((void **)&m->attn_scratch, m->attn_scratch_floats * 4));
     JUNO_TRY(dev_alloc((void **)&m->rope_cs, (size_t)B * (hd / 2) * sizeof(float2)));
-    JUNO_TRY(dev_alloc((void **)&m->d_step, (size_t)4 * B * 4));
-    JUNO_TRY(dev_alloc((void **)&m->d_argmax, (size_t)B * 4));
-    JUNO_TRY(dev_alloc((void **)&m->d_pidx, (size_t)B * kArgmaxBlocks * 4));
-    JUNO_TRY(dev_alloc((void **)&m->d_pval, (size_t)B * kArgmaxBlocks * 4));
-    JUNO_TRY(dev_alloc((void **)&m->d_step_counter, 4));
-    JUNO_CUDA_TRY(cudaMallocHost((void **)&m->h_step, (size_t)4 * B * 4));
+    JUNO_TRY(alloc_step_buffers(m));
     if (m->world > 1) JUNO_TRY(tp_push_setup(m));
     m->finalized = true;
     return JUNO_OK;
@@ -1073,35 +1076,10 @@ static int enqueue_layers_q(juno_model *m, int n, const int32_t *d_slot, const i
     return JUNO_OK;
 }
 
-static int enqueue_step(juno_model *m, int n, int n_splits, bool greedy_advance, bool want_logits, cudaStream_t st) {
+// The greedy pick of n rows of logits and, in the device-side loop, the step to the next position.
+static int enqueue_pick(juno_model *m, int n, bool greedy_advance, bool want_logits, cudaStream_t st) {
     juno_ctx *c = m->ctx;
     const juno_model_cfg &f = m->cfg;
-    const int H = f.hidden, hd = m->hd, B = f.max_batch;
-    const int32_t *d_tok = m->d_step, *d_pos = m->d_step + B, *d_slot = m->d_step + 2 * B, *d_len = m->d_step + 3 * B;
-    if (m->tp_push) {
-        epoch_kernel<<<1, 1, 0, st>>>(m->tp_epoch);
-        JUNO_CUDA_TRY(cudaGetLastError());
-        c->kernel_launches++;
-    }
-    // embedding lookup -> x[0]
-    {
-        juno_qmat *e = m->tok_embd;
-        dim3 grid((H + 255) / 256, n);
-        int64_t rb = e->tiled ? 0 : e->cols / raw_block_elems(e->type) * raw_block_bytes(e->type);
-        embed_kernel<<<grid, 256, 0, st>>>(e->type, e->tiled, e->dev, e->nb, rb, H, f.vocab, d_tok, m->x[0]);
-        JUNO_CUDA_TRY(cudaGetLastError());
-        c->kernel_launches++;
-    }
-    JUNO_TRY(launch_rope_table(c, d_pos, n, hd, f.rope_theta, m->rope_cs, st));
-    int cur = 0;          // x[cur] holds the residual stream
-    // 9..64 sequences: one pass over the weights per product on the FP16 tensor-core kernels; otherwise the exact
-    // integer-MMA GEMV (batches above 64 in chunks of up to eight sequences per pass)
-    const bool batched = n >= m->batched_from && n <= kGemmMaxBatch;
-    if (batched)
-        JUNO_TRY(enqueue_layers_batched(m, n, d_slot, d_len, n_splits, cur, st));
-    else
-        JUNO_TRY(enqueue_layers_q(m, n, d_slot, d_len, n_splits, cur, st));
-    m->last_x = cur;
     LogitsView lv;
     lv.n = n;
     lv.vocab = f.vocab;
@@ -1141,12 +1119,55 @@ static int enqueue_step(juno_model *m, int n, int n_splits, bool greedy_advance,
         c->kernel_launches += 2;
     }
     if (greedy_advance) {
-        advance_kernel<<<1, std::max(32, (n + 31) / 32 * 32), 0, st>>>(n, m->d_argmax, m->d_step, m->d_step + B,
-                                                                      m->d_step + 3 * B, m->d_out_ids, m->d_step_counter);
+        advance_kernel<<<1, std::max(32, (n + 31) / 32 * 32), 0, st>>>(n, m->d_argmax, m->d_step, m->d_step + m->step_cap,
+                                                                      m->d_step + 3 * m->step_cap, m->d_out_ids, m->d_step_counter);
         JUNO_CUDA_TRY(cudaGetLastError());
         c->kernel_launches++;
     }
     return JUNO_OK;
+}
+
+static int enqueue_step(juno_model *m, int n, int n_splits, bool greedy_advance, bool want_logits, cudaStream_t st) {
+    juno_ctx *c = m->ctx;
+    const juno_model_cfg &f = m->cfg;
+    const int H = f.hidden, hd = m->hd, B = m->step_cap;
+    const int32_t *d_tok = m->d_step, *d_pos = m->d_step + B, *d_slot = m->d_step + 2 * B, *d_len = m->d_step + 3 * B;
+    if (m->stack) {
+        RowSet rows;
+        rows.n = n;
+        rows.tokens = d_tok;
+        rows.positions = d_pos;
+        rows.slots = d_slot;
+        rows.lens = d_len;
+        JUNO_TRY(stack_enqueue_layers(c, m->stack, m->pool, rows, n_splits, f.max_ctx, st));
+        JUNO_TRY(stack_enqueue_logits(c, m->stack, nullptr, n, m->logits_loc, st));
+        return enqueue_pick(m, n, greedy_advance, want_logits, st);
+    }
+    if (m->tp_push) {
+        epoch_kernel<<<1, 1, 0, st>>>(m->tp_epoch);
+        JUNO_CUDA_TRY(cudaGetLastError());
+        c->kernel_launches++;
+    }
+    // embedding lookup -> x[0]
+    {
+        juno_qmat *e = m->tok_embd;
+        dim3 grid((H + 255) / 256, n);
+        int64_t rb = e->tiled ? 0 : e->cols / raw_block_elems(e->type) * raw_block_bytes(e->type);
+        embed_kernel<<<grid, 256, 0, st>>>(e->type, e->tiled, e->dev, e->nb, rb, H, f.vocab, d_tok, m->x[0]);
+        JUNO_CUDA_TRY(cudaGetLastError());
+        c->kernel_launches++;
+    }
+    JUNO_TRY(launch_rope_table(c, d_pos, n, hd, f.rope_theta, m->rope_cs, st));
+    int cur = 0;          // x[cur] holds the residual stream
+    // 9..64 sequences: one pass over the weights per product on the FP16 tensor-core kernels; otherwise the exact
+    // integer-MMA GEMV (batches above 64 in chunks of up to eight sequences per pass)
+    const bool batched = n >= m->batched_from && n <= kGemmMaxBatch;
+    if (batched)
+        JUNO_TRY(enqueue_layers_batched(m, n, d_slot, d_len, n_splits, cur, st));
+    else
+        JUNO_TRY(enqueue_layers_q(m, n, d_slot, d_len, n_splits, cur, st));
+    m->last_x = cur;
+    return enqueue_pick(m, n, greedy_advance, want_logits, st);
 }
 
 // Runs one step: the first call for a (n, splits, mode) key runs eagerly (it also sizes every scratch
@@ -1276,7 +1297,9 @@ static int step_check(juno_model *m) {
     if (code) {
         *reinterpret_cast<volatile unsigned *>(c->gemv_scratch.qerr_host) = 0u;
         if (m->tp_failed) cudaMemset(m->tp_failed, 0, 4);
-        if ((code & 0xffu) >= 3u)
+        if ((code & 0xffu) == kErrStackWait)
+            set_error("a matrix product gave up waiting inside a kernel (stage %u of block %u)", (code >> 8) & 0xffu, code >> 16);
+        else if ((code & 0xffu) >= 3u)
             set_error("tensor-parallel rank %u did not deliver its %s within a second (this rank gave up waiting)", (code >> 8) & 0xffu,
                       (code & 0xffu) == 3u ? "partial products" : "greedy pick");
         else
@@ -1296,9 +1319,9 @@ static int bucket_len(int len) {
 static int prepare_step(juno_model *m, int n, juno_seq *const *seqs, const int32_t *tokens, const int32_t *positions,
                         int extra_positions, int *n_splits) {
     juno_ctx *c = m->ctx;
-    const int B = m->cfg.max_batch;
+    const int B = m->step_cap;
     JUNO_REQUIRE(m->finalized, "model is not finalized");
-    JUNO_REQUIRE(n >= 1 && n <= B, "n=%d outside [1, max_batch=%d]", n, B);
+    JUNO_REQUIRE(n >= 1 && n <= m->cfg.max_batch, "n=%d outside [1, max_batch=%d]", n, m->cfg.max_batch);
     JUNO_REQUIRE(seqs && tokens && positions, "null argument");
     int max_len = 0;
     for (int i = 0; i < n; i++) {
@@ -1310,6 +1333,7 @@ static int prepare_step(juno_model *m, int n, juno_seq *const *seqs, const int32
         // a position beyond the sequence's length would make attention read cache rows that were never written
         // (pages come back from the free list as they were left)
         JUNO_REQUIRE(positions[i] <= s->len, "sequence %d: position %d leaves a gap after its %d cached positions", i, positions[i], s->len);
+        JUNO_TRY(seq_resume_check(m->pool, s->len, positions[i]));
         JUNO_TRY(seq_reserve(s, positions[i], positions[i] + 1 + extra_positions, c->stream));
         m->h_step[i] = tokens[i];
         m->h_step[B + i] = positions[i];
@@ -1320,9 +1344,111 @@ static int prepare_step(juno_model *m, int n, juno_seq *const *seqs, const int32
     m->step_kv_bytes = 0;
     for (int i = 0; i < n; i++)
         m->step_kv_bytes += (double)(positions[i] + 1) * m->kv_loc * m->hd * 2 * m->pool->elem_bytes;
-    *n_splits = attn_pick_splits(c, n, m->kv_loc, bucket_len(max_len));
+    *n_splits = m->stack ? stack_pick_splits(c, m->stack, n, bucket_len(max_len)) : attn_pick_splits(c, n, m->kv_loc, bucket_len(max_len));
     JUNO_CUDA_TRY(cudaMemcpyAsync(m->d_step, m->h_step, (size_t)4 * B * 4, cudaMemcpyHostToDevice, c->stream));
     c->h2d_bytes += 4 * n * 4;
+    return JUNO_OK;
+}
+
+// A portion of ONE sequence in passes of as many positions as the model's kernels take at once.  want[0..n_want): places
+// in the portion whose logits go to logits_host, in that order; argmax_out (optional): the greedy pick at the last of them.
+static int prefill_run(juno_model *m, juno_seq *seq, const int32_t *token_ids, int n_tokens, int start_pos, int n_want, const int32_t *want,
+                       float *logits_host, int32_t *argmax_out) {
+    JUNO_TRY(model_check(m));
+    juno_ctx *c = m->ctx;
+    std::lock_guard<std::recursive_mutex> lk(c->mu);
+    DeviceGuard g(c->device);
+    JUNO_REQUIRE(m->finalized, "model is not finalized");
+    JUNO_REQUIRE(seq && seq->magic == kMagicSeq && seq->pool == m->pool, "sequence is closed or belongs to another model");
+    JUNO_REQUIRE(token_ids && n_tokens >= 1 && start_pos >= 0, "bad prefill arguments (n_tokens=%d, start_pos=%d)", n_tokens, start_pos);
+    JUNO_REQUIRE(start_pos + n_tokens <= m->cfg.max_ctx, "position %d is beyond max_ctx %d", start_pos + n_tokens - 1, m->cfg.max_ctx);
+    JUNO_REQUIRE(start_pos <= seq->len, "start position %d leaves a gap after the %d cached positions", start_pos, seq->len);
+    JUNO_TRY(seq_resume_check(m->pool, seq->len, start_pos));
+    const juno_model_cfg &f = m->cfg;
+    const int B = m->step_cap, chunk_max = m->stack ? B : std::min(B, kGemmMaxBatch), V = f.vocab;
+    JUNO_REQUIRE(n_want == 0 || !m->vocab_sharded, "prefill logits are not implemented for a sharded vocabulary");
+    cudaStream_t st = c->stream;
+    for (int done = 0; done < n_tokens;) {
+        const int n = std::min(chunk_max, n_tokens - done), pos0 = start_pos + done;
+        JUNO_TRY(step_sync(m));  // the pinned step buffer is reused
+        JUNO_TRY(seq_reserve(seq, pos0, pos0 + n, st));
+        for (int i = 0; i < n; i++) {
+            m->h_step[i] = token_ids[done + i];
+            m->h_step[B + i] = pos0 + i;
+            m->h_step[2 * B + i] = seq->slot;
+            m->h_step[3 * B + i] = pos0 + i + 1;
+        }
+        JUNO_CUDA_TRY(cudaMemcpyAsync(m->d_step, m->h_step, (size_t)4 * B * 4, cudaMemcpyHostToDevice, st));
+        c->h2d_bytes += 4 * n * 4;
+        std::vector<std::pair<int, int>> rows;  // (row of this pass, index into want)
+        for (int k = 0; k < n_want; k++)
+            if (want[k] >= done && want[k] < done + n) rows.emplace_back(want[k] - done, k);
+        const int32_t *d_tok = m->d_step, *d_pos = m->d_step + B, *d_slot = m->d_step + 2 * B, *d_len = m->d_step + 3 * B;
+        if (m->stack) {
+            RowSet rs;
+            rs.n = n;
+            rs.one_seq = true;
+            rs.tokens = d_tok;
+            rs.positions = d_pos;
+            rs.slots = d_slot;
+            rs.lens = d_len;
+            JUNO_TRY(stack_enqueue_layers(c, m->stack, m->pool, rs, stack_pick_splits(c, m->stack, n, pos0 + n), pos0 + n, st));
+        } else {
+            m->step_kv_bytes = 0;
+            for (int i = 0; i < n; i++) m->step_kv_bytes += (double)(pos0 + i + 1) * m->kv_loc * m->hd * 2 * m->pool->elem_bytes;
+            const int n_splits = attn_pick_splits(c, n, m->kv_loc, bucket_len(pos0 + n));
+            juno_qmat *e = m->tok_embd;
+            dim3 grid((f.hidden + 255) / 256, n);
+            int64_t rb = e->tiled ? 0 : e->cols / raw_block_elems(e->type) * raw_block_bytes(e->type);
+            embed_kernel<<<grid, 256, 0, st>>>(e->type, e->tiled, e->dev, e->nb, rb, f.hidden, V, d_tok, m->x[0]);
+            JUNO_CUDA_TRY(cudaGetLastError());
+            c->kernel_launches++;
+            JUNO_TRY(launch_rope_table(c, d_pos, n, m->hd, f.rope_theta, m->rope_cs, st));
+            int cur = 0;
+            JUNO_TRY(enqueue_layers_batched(m, n, d_slot, d_len, n_splits, cur, st, d_pos, !rows.empty()));
+            m->last_x = cur;
+        }
+        m->last_n = n;
+        c->forward_calls++;
+        for (size_t i0 = 0; i0 < rows.size();) {
+            // a stack computes the wanted rows only, as many as the buffer holds at a time; the quantised layers have computed all
+            size_t i1 = m->stack ? std::min(rows.size(), i0 + (size_t)m->logit_cap) : rows.size();
+            if (m->stack) {
+                std::vector<int32_t> idx;
+                for (size_t i = i0; i < i1; i++) idx.push_back(rows[i].first);
+                JUNO_CUDA_TRY(cudaMemcpyAsync(m->stack->row_idx, idx.data(), idx.size() * 4, cudaMemcpyHostToDevice, st));
+                JUNO_TRY(stack_enqueue_logits(c, m->stack, m->stack->row_idx, (int)idx.size(), m->logits_loc, st));
+            }
+            for (size_t i = i0; i < i1;) {
+                const int src = m->stack ? (int)(i - i0) : rows[i].first;
+                size_t run = 1;  // rows that lie side by side at both ends travel as one copy
+                while (i + run < i1 && rows[i + run].second == rows[i].second + (int)run && (m->stack || rows[i + run].first == src + (int)run)) run++;
+                if (logits_host) {
+                    JUNO_CUDA_TRY(cudaMemcpyAsync(logits_host + (size_t)rows[i].second * V, m->logits_loc + (size_t)src * m->vocab_loc, run * V * 4, cudaMemcpyDeviceToHost, st));
+                    c->d2h_bytes += (int64_t)run * V * 4;
+                }
+                i += run;
+            }
+            if (argmax_out && i1 == rows.size()) {
+                LogitsView lv;
+                lv.n = 1;
+                lv.vocab = V;
+                lv.base = m->logits_loc + (size_t)(m->stack ? i1 - 1 - i0 : rows[i1 - 1].first) * m->vocab_loc;
+                lv.vloc = V;
+                argmax_partial_kernel<<<dim3(kArgmaxBlocks, 1), 256, 0, st>>>(lv, m->d_pval, m->d_pidx);
+                argmax_final_kernel<<<1, 64, 0, st>>>(m->d_pval, m->d_pidx, 1, m->d_argmax);
+                JUNO_CUDA_TRY(cudaGetLastError());
+                c->kernel_launches += 2;
+                JUNO_CUDA_TRY(cudaMemcpyAsync(argmax_out, m->d_argmax, 4, cudaMemcpyDeviceToHost, st));
+                c->d2h_bytes += 4;
+            }
+            i0 = i1;
+        }
+        done += n;
+    }
+    JUNO_TRY(step_sync(m));
+    JUNO_TRY(step_check(m));
+    seq->len = std::max(seq->len, start_pos + n_tokens);
     return JUNO_OK;
 }
 
@@ -1380,78 +1506,15 @@ int juno_forward(juno_model *m, int32_t n, juno_seq *const *seqs, const int32_t 
 
 int juno_prefill(juno_model *m, juno_seq *seq, const int32_t *token_ids, int32_t n_tokens, int32_t start_pos,
                  float *logits_host, int32_t *argmax_out) {
-    JUNO_TRY(model_check(m));
-    juno_ctx *c = m->ctx;
-    std::lock_guard<std::recursive_mutex> lk(c->mu);
-    DeviceGuard g(c->device);
-    JUNO_REQUIRE(m->finalized, "model is not finalized");
-    JUNO_REQUIRE(seq && seq->magic == kMagicSeq && seq->pool == m->pool, "sequence is closed or belongs to another model");
-    JUNO_REQUIRE(token_ids && n_tokens >= 1 && start_pos >= 0, "bad prefill arguments (n_tokens=%d, start_pos=%d)", n_tokens, start_pos);
-    JUNO_REQUIRE(start_pos + n_tokens <= m->cfg.max_ctx, "position %d is beyond max_ctx %d", start_pos + n_tokens - 1, m->cfg.max_ctx);
-    JUNO_REQUIRE(start_pos <= seq->len, "start position %d leaves a gap after the %d cached positions", start_pos, seq->len);
-    JUNO_REQUIRE(m->pool->dtype == 0 || m->pool->dtype == 1, "unsupported KV type");
-    const juno_model_cfg &f = m->cfg;
-    const int B = f.max_batch, chunk_max = std::min(B, kGemmMaxBatch), V = f.vocab;
-    cudaStream_t st = c->stream;
-    for (int done = 0; done < n_tokens;) {
-        const int n = std::min(chunk_max, n_tokens - done), pos0 = start_pos + done;
-        const bool last = done + n == n_tokens;
-        JUNO_TRY(step_sync(m));  // the pinned step buffer is reused
-        JUNO_TRY(seq_reserve(seq, pos0, pos0 + n, st));
-        for (int i = 0; i < n; i++) {
-            m->h_step[i] = token_ids[done + i];
-            m->h_step[B + i] = pos0 + i;
-            m->h_step[2 * B + i] = seq->slot;
-            m->h_step[3 * B + i] = pos0 + i + 1;
-        }
-        JUNO_CUDA_TRY(cudaMemcpyAsync(m->d_step, m->h_step, (size_t)4 * B * 4, cudaMemcpyHostToDevice, st));
-        c->h2d_bytes += 4 * n * 4;
-        m->step_kv_bytes = 0;
-        for (int i = 0; i < n; i++) m->step_kv_bytes += (double)(pos0 + i + 1) * m->kv_loc * m->hd * 2 * m->pool->elem_bytes;
-        const int n_splits = attn_pick_splits(c, n, m->kv_loc, bucket_len(pos0 + n));
-        const int32_t *d_tok = m->d_step, *d_pos = m->d_step + B, *d_slot = m->d_step + 2 * B, *d_len = m->d_step + 3 * B;
-        {
-            juno_qmat *e = m->tok_embd;
-            dim3 grid((f.hidden + 255) / 256, n);
-            int64_t rb = e->tiled ? 0 : e->cols / raw_block_elems(e->type) * raw_block_bytes(e->type);
-            embed_kernel<<<grid, 256, 0, st>>>(e->type, e->tiled, e->dev, e->nb, rb, f.hidden, V, d_tok, m->x[0]);
-            JUNO_CUDA_TRY(cudaGetLastError());
-            c->kernel_launches++;
-        }
-        JUNO_TRY(launch_rope_table(c, d_pos, n, m->hd, f.rope_theta, m->rope_cs, st));
-        int cur = 0;
-        JUNO_TRY(enqueue_layers_batched(m, n, d_slot, d_len, n_splits, cur, st, d_pos, last && (logits_host || argmax_out)));
-        m->last_x = cur;
-        m->last_n = n;
-        c->forward_calls++;
-        if (last && (logits_host || argmax_out)) {
-            // row n-1 is the last prompt position
-            const float *row = m->logits_loc + (size_t)(n - 1) * m->vocab_loc;
-            JUNO_REQUIRE(!m->vocab_sharded, "prefill logits are not implemented for a sharded vocabulary");
-            if (argmax_out) {
-                LogitsView lv;
-                lv.n = 1;
-                lv.vocab = V;
-                lv.base = row;
-                lv.vloc = V;
-                argmax_partial_kernel<<<dim3(kArgmaxBlocks, 1), 256, 0, st>>>(lv, m->d_pval, m->d_pidx);
-                argmax_final_kernel<<<1, 64, 0, st>>>(m->d_pval, m->d_pidx, 1, m->d_argmax);
-                JUNO_CUDA_TRY(cudaGetLastError());
-                c->kernel_launches += 2;
-                JUNO_CUDA_TRY(cudaMemcpyAsync(argmax_out, m->d_argmax, 4, cudaMemcpyDeviceToHost, st));
-                c->d2h_bytes += 4;
-            }
-            if (logits_host) {
-                JUNO_CUDA_TRY(cudaMemcpyAsync(logits_host, row, (size_t)V * 4, cudaMemcpyDeviceToHost, st));
-                c->d2h_bytes += (int64_t)V * 4;
-            }
-        }
-        done += n;
-    }
-    JUNO_TRY(step_sync(m));
-    JUNO_TRY(step_check(m));
-    seq->len = std::max(seq->len, start_pos + n_tokens);
-    return JUNO_OK;
+    const int32_t last = n_tokens - 1;
+    return prefill_run(m, seq, token_ids, n_tokens, start_pos, logits_host || argmax_out ? 1 : 0, &last, logits_host, argmax_out);
+}
+
+int juno_prefill_logits(juno_model *m, juno_seq *seq, const int32_t *token_ids, int32_t n_tokens, int32_t start_pos, int32_t n_want,
+                        const int32_t *want, float *logits_host) {
+    JUNO_REQUIRE(n_want >= 0 && (n_want == 0 || (want && logits_host)), "bad prefill arguments (n_want=%d)", n_want);
+    for (int i = 0; i < n_want; i++) JUNO_REQUIRE(want[i] >= 0 && want[i] < n_tokens, "wanted place %d outside the %d tokens", want[i], n_tokens);
+    return prefill_run(m, seq, token_ids, n_tokens, start_pos, n_want, want, logits_host, nullptr);
 }
 
 int juno_decode_greedy(juno_model *m, int32_t n, juno_seq *const *seqs, const int32_t *first_tokens,
@@ -1499,8 +1562,9 @@ int juno_model_last_hidden(juno_model *m, int32_t n, float *hidden_host) {
     juno_ctx *c = m->ctx;
     std::lock_guard<std::recursive_mutex> lk(c->mu);
     DeviceGuard g(c->device);
-    JUNO_CUDA_TRY(cudaMemcpyAsync(hidden_host, m->x[m->last_x], (size_t)n * m->cfg.hidden * 4, cudaMemcpyDeviceToHost,
-                                  c->stream));
+    const float *x = m->stack ? stack_residual(m->stack) : m->x[m->last_x];
+    const size_t row = (size_t)m->cfg.hidden * 4, pitch = m->stack ? (size_t)m->stack->spec.wp() * 4 : row;
+    JUNO_CUDA_TRY(cudaMemcpy2DAsync(hidden_host, row, x, pitch, row, (size_t)n, cudaMemcpyDeviceToHost, c->stream));
     JUNO_CUDA_TRY(cudaStreamSynchronize(c->stream));
     return JUNO_OK;
 }
@@ -1547,6 +1611,27 @@ int juno_model_tp_mode(juno_model *m, int32_t *mode) {
     JUNO_TRY(model_check(m));
     JUNO_REQUIRE(mode, "mode is null");
     *mode = m->world <= 1 ? 0 : (m->tp_push ? 2 : 1);
+    return JUNO_OK;
+}
+
+int juno_model_describe(juno_model *m, juno_model_info *info) {
+    JUNO_TRY(model_check(m));
+    JUNO_REQUIRE(info, "info is null");
+    memset(info, 0, sizeof(*info));
+    snprintf(info->architecture, sizeof(info->architecture), "%s", m->architecture.c_str());
+    info->hidden = m->cfg.hidden;
+    info->n_layers = m->cfg.n_layers;
+    info->vocab = m->cfg.vocab;
+    info->max_batch = m->cfg.max_batch;
+    info->max_seqs = m->cfg.max_seqs;
+    info->max_ctx = m->cfg.max_ctx;
+    info->max_rows = m->stack ? m->step_cap : std::min(m->step_cap, kGemmMaxBatch);
+    info->weight_bytes = m->stack ? (int64_t)m->stack->weight_bytes : 0;
+    if (m->pool) {
+        info->cache_bytes_per_token = m->pool->latent ? 0 : (int64_t)2 * m->pool->n_layers * m->pool->n_kv_heads * m->pool->head_dim * m->pool->elem_bytes;
+        for (int w : m->pool->row_width) info->cache_bytes_per_token += (int64_t)w * m->pool->elem_bytes;
+        info->state_bytes_per_seq = (int64_t)m->pool->n_layers * m->pool->state_ring * m->pool->state_width * 4;
+    }
     return JUNO_OK;
 }
 

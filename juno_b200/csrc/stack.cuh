@@ -1,0 +1,110 @@
+// Layer stacks with dense (BF16 or FP32) weights: the description a model design is turned into, its weights in device
+// memory, and the passes that run it.  A design (csrc/vosotar.cu) parses its configuration into a StackSpec and loads its
+// tensors; everything below is shared between designs that use the same mechanisms.
+#pragma once
+#include <string>
+#include <vector>
+
+#include "gemm_rows.cuh"
+#include "latent_attn.cuh"
+#include "rowops.cuh"
+#include "safetensors.cuh"
+
+namespace juno {
+
+// Latent attention without positions: queries through a normed latent of q_rank, keys and values through a normed latent of
+// kv_rank that alone is cached; one sigmoid gate per head on the output.
+struct LatentMixerSpec {
+    int heads = 0, dim = 0, vdim = 0, q_rank = 0, kv_rank = 0;
+    float scale = 0.f;
+    // padded sizes of the device layouts (multiples of 16: tensor-core steps and 32-byte rows)
+    int qp() const { return pad16(q_rank); }
+    int rp() const { return pad16(kv_rank); }
+    int dp() const { return pad16(dim); }
+    int vp() const { return pad16(vdim); }
+    int kv_col() const { return qp(); }
+    int gate_col() const { return qp() + rp(); }
+    int down_rows() const { return qp() + rp() + pad16(heads); }
+};
+
+struct StackLayerSpec {
+    LatentMixerSpec mix;
+    int ff = 0;            // 0: no feed-forward
+    int weights_of = -1;   // >= 0: this layer runs with that layer's weights
+};
+
+struct StackSpec {
+    int width = 0, vocab = 0, taps = 1;
+    float eps = 0.f;
+    std::vector<StackLayerSpec> layers;
+    int wp() const { return pad16(width); }
+    int weights(int layer) const {
+        while (layers[layer].weights_of >= 0) layer = layers[layer].weights_of;
+        return layer;
+    }
+};
+
+struct StackMat {
+    void *w = nullptr;
+    int rows = 0, cols = 0;  // padded; cols is also the row pitch
+};
+
+struct StackLayerWeights {
+    float norm1 = 0, norm1b = 0, norm2 = 0, norm2b = 0;  // norms with one number
+    StackMat down;    // W_dq | W_dkv | W_g, one product on the convolved input
+    StackMat uq, ukt, ukv, o;  // ukt: per head W_uk transposed [rank][dim]; ukv: W_uk over W_uv
+    StackMat rg1, rg2, up, mdown;
+    float *dq_norm = nullptr, *dkv_norm = nullptr, *rg1_b = nullptr, *rg2_b = nullptr;
+    void *conv = nullptr;  // [taps][wp]
+};
+
+struct StackNet {
+    StackSpec spec;
+    int dt = DT_BF16;
+    StackMat embed, head;
+    float embed_norm = 0, final_norm = 0;
+    std::vector<StackLayerWeights> layers;  // entries of layers with weights_of stay empty
+    std::vector<void *> owned;              // every device allocation
+    // buffers of a pass
+    int cap = 0, lat_cap = 0, logit_cap = 0;
+    float *x = nullptr, *u = nullptr, *row_scale = nullptr;
+    float *x2 = nullptr;
+    void *h = nullptr, *hc = nullptr, *gate = nullptr, *z = nullptr, *cq = nullptr, *q = nullptr, *qlat = nullptr, *olat = nullptr,
+         *att = nullptr, *act = nullptr, *fin = nullptr;
+    int ldu = 0, ldcq = 0, ldq = 0, ldlat = 0, ldatt = 0, ldact = 0;
+    int32_t *row_idx = nullptr;  // device list of rows whose logits are wanted
+    double weight_bytes = 0;     // bytes a one-token step reads
+    int last_x = 0;
+};
+
+// ── loading ──
+// Host image of a padded matrix, filled block by block and uploaded once.
+struct HostMat {
+    int dt, rows, cols;
+    std::vector<uint8_t> data;
+    HostMat(int dtype, int r, int c) : dt(dtype), rows(r), cols(c), data((size_t)r * c * dt_bytes(dtype), 0) {}
+    // dst[row + i][col + j] = src[r0 + i][c0 + j]
+    void put(const juno_safetensors *f, const StTensor &t, int64_t r0, int64_t c0, int nr, int nc, int row, int col);
+    // dst[row + j][col + i] = src[r0 + i][c0 + j]
+    void put_transposed(const juno_safetensors *f, const StTensor &t, int64_t r0, int64_t c0, int nr, int nc, int row, int col);
+};
+int stack_upload(juno_ctx *c, StackNet *net, const HostMat &m, StackMat *out);
+int stack_upload_f32(juno_ctx *c, StackNet *net, const std::vector<float> &v, float **out);
+float st_value(const juno_safetensors *f, const StTensor &t, int64_t i);
+
+// ── running ──
+int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int logit_rows);
+void stack_free(StackNet *net);
+// All layers for `rows`; `len_bound` bounds positions + 1 over the rows.  The residual stream ends in the net's x.
+int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, cudaStream_t st);
+// logits[i] = head . norm(x[row_idx[i]]) (row_idx null: row i), n rows
+int stack_enqueue_logits(juno_ctx *c, StackNet *net, const int32_t *row_idx, int n, float *logits, cudaStream_t st);
+const float *stack_residual(const StackNet *net);  // residual stream of the last pass, rows of wp() floats
+int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bound);
+
+// ── designs ──
+struct Json;
+int vosotar_spec(const Json &cfg, StackSpec *spec);
+int vosotar_load(juno_ctx *c, const juno_safetensors *f, const StackSpec &spec, int dt, StackNet **out);
+
+}  // namespace juno

@@ -68,8 +68,24 @@ class TensorShardContext:
         return self.hidden_dim // self.tensor_world_size
 
 
+@dataclass
+class ModelShape:
+    """What a handler knows about a model that the registry opened (juno_model_describe)."""
+    architecture: str
+    hidden: int
+    n_layers: int
+    vocab: int
+    max_batch: int
+    max_ctx: int
+    max_rows: int
+    weight_bytes: int
+    cache_bytes_per_token: int
+    state_bytes_per_seq: int
+
+
 class B200TransformerHandler:
-    """LLaMA-family decode on one B200 (or one tensor-parallel rank)."""
+    """Decode on one B200 (or one tensor-parallel rank): the LLaMA family from tensors or GGUF, and every design of the model
+    registry from its file or folder (`open`)."""
 
     def __init__(self, arch: synth.Arch, ctx: GpuContext | None = None, max_batch: int = 1, max_seqs: int = 8,
                  max_ctx: int = 2048, kv_dtype: str = "f16", tp_rank: int = 0, tp_world: int = 1,
@@ -94,6 +110,24 @@ class B200TransformerHandler:
         self.max_batch = max_batch
         self._seqs: dict[str, C.c_void_p] = {}
         self._released = False
+
+    @classmethod
+    def open(cls, path, ctx: GpuContext | None = None, max_batch: int = 1, max_seqs: int = 8, max_ctx: int = 2048,
+             dtype: str = "default", max_rows: int = 0) -> "B200TransformerHandler":
+        """Opens whatever the path holds (juno_model_open): a folder with config.json and model.safetensors whose architecture
+        is registered, or a GGUF file.  dtype "default" or "f32" (true 32-bit); max_rows: prompt positions per pass."""
+        self = cls.__new__(cls)
+        self.ctx = ctx or GpuContext.shared(0)
+        self._L = self.ctx._L
+        o = _lib.OpenOpts(C.sizeof(_lib.OpenOpts), max_batch, max_seqs, max_ctx, {"default": 0, "f32": 1}[dtype], max_rows)
+        h = C.c_void_p()
+        check(self._L.juno_model_open(self.ctx.handle, str(path).encode(), C.byref(o), C.byref(h)), "juno_model_open")
+        self.handle, self.max_batch, self._seqs, self._released = h, max_batch, {}, False
+        i = _lib.ModelInfo()
+        check(self._L.juno_model_describe(h, C.byref(i)), "juno_model_describe")
+        self.arch = ModelShape(i.architecture.decode(), i.hidden, i.n_layers, i.vocab, i.max_batch, i.max_ctx, i.max_rows,
+                               i.weight_bytes, i.cache_bytes_per_token, i.state_bytes_per_seq)
+        return self
 
     @staticmethod
     def nccl_unique_id() -> bytes:
@@ -174,6 +208,36 @@ class B200TransformerHandler:
         check(self._L.juno_prefill(self.handle, self._seq(request_id), _ptr(toks), len(toks), int(start_pos),
                                    _ptr(logits) if want_logits else None, None), "juno_prefill")
         return logits
+
+    def prefill_logits(self, request_id: str, token_ids, start_pos: int = 0, want=()) -> np.ndarray:
+        """One portion of a prompt (juno_prefill_logits): logits [len(want), vocab] at the given places of the portion."""
+        toks = np.ascontiguousarray(np.asarray(token_ids, dtype=np.int32))
+        idx = np.ascontiguousarray(np.asarray(list(want), dtype=np.int32))
+        logits = np.empty((len(idx), self.arch.vocab), dtype=np.float32)
+        check(self._L.juno_prefill_logits(self.handle, self._seq(request_id), _ptr(toks), len(toks), int(start_pos), len(idx), _ptr(idx),
+                                          _ptr(logits)), "juno_prefill_logits")
+        return logits
+
+    def length(self, request_id: str) -> int:
+        """Positions the request has cached so far."""
+        s = self._seqs.get(request_id)
+        if s is None:
+            return 0
+        n = C.c_int32()
+        check(self._L.juno_seq_length(s, C.byref(n)), "juno_seq_length")
+        return n.value
+
+    def feed(self, request_id: str, token_ids, want=()) -> np.ndarray:
+        """The next tokens of a request, continuing from its cache and state: a single token takes the decode step, more take
+        the prompt path.  Returns the logits at the places `want` of these tokens."""
+        pos = self.length(request_id)
+        if len(token_ids) > 1:
+            return self.prefill_logits(request_id, token_ids, pos, want)
+        if len(want):
+            row = self.forward_batch([request_id], [[token_ids[0]]], [pos])
+            return np.repeat(row, len(want), axis=0)
+        self.forward_batch([request_id], [[token_ids[0]]], [pos], want_logits=False, want_argmax=True)
+        return np.empty((0, self.arch.vocab), dtype=np.float32)
 
     def decode_greedy(self, request_ids, first_tokens, positions, steps: int) -> np.ndarray:
         """`steps` greedy tokens per request with the loop kept on the device; returns [steps, n] ids."""
