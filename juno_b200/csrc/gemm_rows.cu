@@ -1,11 +1,9 @@
-// Matrix products of many rows.  FP32 runs on the FMA units in true 32-bit (no reduced-precision matrix mode).
+// Matrix products of many rows.  BF16 runs on the tensor cores (gemm_rows_tc.cu); FP32 runs on the FMA units in true 32-bit (no reduced-precision matrix mode).
 #include "gemm_rows.cuh"
 
 #include <algorithm>
 
 namespace juno {
-
-using bf16 = __nv_bfloat16;
 
 constexpr int kSimtTile = 64, kSimtK = 16;
 
@@ -64,17 +62,14 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const GemmArgs p) {
 }
 
 int launch_gemm_rows(juno_ctx *c, int dt, const GemmArgs &a, unsigned *err, cudaStream_t st) {
-    (void)err;
     JUNO_REQUIRE(a.a && a.w && a.out && a.M > 0 && a.N > 0 && a.K > 0 && a.K % 16 == 0 && a.lda % 16 == 0 && a.ldw % 16 == 0 && a.a_step % 16 == 0 && a.groups >= 1,
                  "matrix product: bad arguments (M %d, N %d, K %d)", a.M, a.N, a.K);
     const double es = dt_bytes(dt);
     const double algo = a.groups * ((double)a.M * a.K + (double)a.N * a.K) * es + (double)a.groups * a.M * a.N * (a.epi == GE_F32 ? 4.0 : es);
     ProfScope prof(c, st, PROF_GEMM_ROWS, algo);
+    if (dt == DT_BF16) return launch_gemm_rows_tc(c, a, err, st);
     const dim3 grid((unsigned)((a.N + kSimtTile - 1) / kSimtTile), (unsigned)((a.M + kSimtTile - 1) / kSimtTile), (unsigned)a.groups);
-    if (dt == DT_F32)
-        gemm_simt_kernel<float><<<grid, 256, 0, st>>>(a);
-    else
-        gemm_simt_kernel<bf16><<<grid, 256, 0, st>>>(a);
+    gemm_simt_kernel<float><<<grid, 256, 0, st>>>(a);
     JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;

@@ -28,9 +28,9 @@ struct GemmArgs {
     const void *aux = nullptr;
     int ldaux = 0;
     int groups = 1, a_step = 0, w_step = 0, o_step = 0;
-    int a_rows = 0;  // rows of `a` that may be read (0: M)
     int w_rows = 0;  // rows of `w` in memory (0: N, or w_step * groups)
 };
+int launch_gemm_rows_tc(juno_ctx *c, const GemmArgs &a, unsigned *err, cudaStream_t st);  // BF16, tcgen05
 int launch_gemm_rows(juno_ctx *c, int dt, const GemmArgs &a, unsigned *err, cudaStream_t st);
 
 }  // namespace juno

@@ -148,3 +148,62 @@ def random_model(arch: Arch, seed: int, type_map=q4_k_m_type, norm: str = "ones"
             for kind in (T_ATTN_Q_BIAS, T_ATTN_K_BIAS, T_ATTN_V_BIAS):
                 n = tensor_shape(arch, kind)[1]
                 yield kind, l, F32, 1, n, rng_norm.standard_normal(n).astype(np.float32).view(np.uint8)
+
+
+# ── Vosotar stacks (config.json + BF16 tensors) ──────────────────────────────────────────────────
+def vosotar_config(width: int, vocab: int, layers, taps: int = 4, eps: float = 1e-6) -> dict:
+    """layers: dicts with heads, dim, vdim, q_rank, kv_rank, scale, ff (0 or None: no feed-forward), optional weights_of."""
+    out = []
+    for L in layers:
+        e = {"type": "latent_attention", "mixer": {k: L[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank", "scale")},
+             "mlp": {"kind": "dense", "ff": L["ff"]} if L.get("ff") else None}
+        if L.get("weights_of") is not None:
+            e["weights_of"] = L["weights_of"]
+        out.append(e)
+    return {"architecture": "Vosotar", "width": width, "vocab": vocab, "norm": {"eps": eps}, "canon": {"taps": taps}, "layers": out}
+
+
+def vosotar_shapes(cfg: dict) -> dict:
+    """Tensor name -> (shape, fan-in or None) in file order."""
+    W, V, taps = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
+    t = {"embed": ((V, W), None), "embed.norm": ((), None), "final.norm": ((), None), "head": ((V, W), W)}
+    for i, e in enumerate(cfg["layers"]):
+        if e.get("weights_of") is not None:
+            continue
+        p, m = f"l{i}.", e["mixer"]
+        H, d, dv, qr, kr = m["heads"], m["dim"], m["vdim"], m["q_rank"], m["kv_rank"]
+        t.update({p + "norm1": ((), None), p + "norm1b": ((), None), p + "mix.dq": ((qr, W), W), p + "mix.dq.norm": ((qr,), None),
+                  p + "mix.uq": ((H * d, qr), qr), p + "mix.dkv": ((kr, W), W), p + "mix.dkv.norm": ((kr,), None),
+                  p + "mix.uk": ((H * d, kr), kr), p + "mix.uv": ((H * dv, kr), kr), p + "mix.g": ((H, W), W),
+                  p + "mix.o": ((W, H * dv), H * dv), p + "canon1": ((W, taps), taps), p + "rg1": ((W, W), W), p + "rg1.b": ((W,), None)})
+        if e["mlp"] is not None:
+            ff = e["mlp"]["ff"]
+            t.update({p + "norm2": ((), None), p + "norm2b": ((), None), p + "mlp.up": ((ff, W), W), p + "mlp.down": ((W, ff), ff),
+                      p + "rg2": ((W, W), W), p + "rg2.b": ((W,), None)})
+    return t
+
+
+def random_vosotar(cfg: dict, seed: int, fast: bool = False) -> dict:
+    """Random tensors (BF16 bit patterns) of a configuration: fan-in scaled normals, norm weights round one, biases round zero.
+    fast: large matrices repeat a drawn block (benchmarks, where only the shapes matter)."""
+    from .safetensors_file import to_bf16
+    rng = np.random.default_rng(seed)
+    block = to_bf16(rng.standard_normal(1 << 20)) if fast else None
+    out = {}
+    for name, (shape, fan) in vosotar_shapes(cfg).items():
+        n = int(np.prod(shape)) if shape else 1
+        if fast and n > (1 << 20):
+            scale = int(round(np.log2(fan) / 2)) if fan else 0  # a power of two: an exponent shift of the block
+            b = (block.astype(np.int32) - (scale << 7)).astype(np.uint16) if scale else block
+            out[name] = np.resize(np.roll(b, int(rng.integers(1 << 20))), n).reshape(shape)
+            continue
+        if fan:
+            v = rng.standard_normal(n) / np.sqrt(fan)
+        elif name.endswith(".b"):
+            v = 0.5 * rng.standard_normal(n)
+        elif name == "embed":
+            v = rng.standard_normal(n)
+        else:
+            v = 1.0 + 0.3 * rng.standard_normal(n)
+        out[name] = to_bf16(v).reshape(shape)
+    return out
