@@ -1,0 +1,561 @@
+// BF16 attention over latent pages on the tensor cores: the split kernel of decode steps with its merge, and causal flash
+// attention over expanded keys and values for prompts (see latent_attn.cuh).
+#include <algorithm>
+#include <mutex>
+
+#include "latent_attn.cuh"
+#include "mma_bf16.cuh"
+
+namespace juno {
+
+using bf16 = __nv_bfloat16;
+constexpr float kLog2e = 1.4426950408889634f;
+
+// ───────────────────────────── decode: splits of the context ──────────────────────────────
+// A CTA takes a group of 16 * MT heads of one row and a range of positions, 32 at a time.  Scores: warp (rank quarter, 16
+// positions) multiplies its part of q_lat with the tile, the four quarters are added in shared memory; online softmax by rows;
+// then each warp owns a range of latent columns of O += P C, reading the same tile transposed.
+constexpr int kSpKeys = 32, kSpThreads = 256, kSpWarps = 8;
+
+struct SplitParams {
+    const bf16 *plane;
+    const int32_t *table, *positions, *slots;
+    int max_pages, heads, rank, n_splits;
+    float scale_log2;
+    const bf16 *q;
+    float *part_o, *part_ml;
+};
+
+template <int MT, int NP>  // NP: 16-column pairs of n-tiles a warp owns at most
+__global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_split_kernel(const SplitParams p) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    constexpr int HM = 16 * MT;
+    const int R = p.rank, pitch = R + 8;
+    bf16 *qs = reinterpret_cast<bf16 *>(sm);          // [HM][pitch]
+    bf16 *cs = qs + HM * pitch;                       // [2][kSpKeys][pitch]
+    bf16 *ps = cs + 2 * kSpKeys * pitch;              // [HM][kSpKeys + 8]
+    float *ss = reinterpret_cast<float *>(ps + HM * (kSpKeys + 8));  // [4][HM][kSpKeys + 2]
+    float *fac = ss + 4 * HM * (kSpKeys + 2), *mrow = fac + HM, *lrow = mrow + HM;
+    const int split = blockIdx.x, h0 = blockIdx.y * HM, row = blockIdx.z, nh = min(HM, p.heads - h0);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int len = p.positions[row] + 1;
+    const int tiles = (len + kSpKeys - 1) / kSpKeys, per = (tiles + p.n_splits - 1) / p.n_splits;
+    const int j0 = split * per * kSpKeys, j1 = min(len, j0 + per * kSpKeys);
+    const size_t part = ((size_t)row * p.heads + h0) * p.n_splits + split;  // + head * n_splits
+    if (j0 >= j1) {
+        if (tid < nh) {
+            p.part_ml[(part + (size_t)tid * p.n_splits) * 2] = -INFINITY;
+            p.part_ml[(part + (size_t)tid * p.n_splits) * 2 + 1] = 0.f;
+        }
+        return;
+    }
+    const int32_t *table = p.table + (size_t)p.slots[row] * p.max_pages;
+    const int chunks = R >> 3;
+    auto load_tile = [&](int j, int buf) {
+        bf16 *dst = cs + (size_t)buf * kSpKeys * pitch;
+        for (int i = tid; i < kSpKeys * chunks; i += kSpThreads) {
+            const int r = i / chunks, ch = i - r * chunks;
+            const bool ok = j + r < j1;
+            const bf16 *src = latent_row(p.plane, table, R, ok ? j + r : j0) + ch * 8;
+            cp16(smem_addr(dst + r * pitch + ch * 8), src, ok);
+        }
+        cp_commit();
+    };
+    {
+        const bf16 *q = p.q + ((size_t)row * p.heads + h0) * R;
+        for (int i = tid; i < HM * chunks; i += kSpThreads) {
+            const int r = i / chunks, ch = i - r * chunks;
+            const bool ok = r < nh;
+            cp16(smem_addr(qs + r * pitch + ch * 8), q + (ok ? (size_t)r * R + ch * 8 : 0), ok);
+        }
+    }
+    load_tile(j0, 0);
+    if (tid < HM) {
+        mrow[tid] = -INFINITY;
+        lrow[tid] = 0.f;
+    }
+    const int kg = warp & 1, rq = warp >> 1;                      // 16 positions, quarter of the rank
+    const int ksteps = R >> 4, ks0 = ksteps * rq / 4, ks1 = ksteps * (rq + 1) / 4;
+    const int pairs = R >> 4, pw = (pairs + kSpWarps - 1) / kSpWarps, c0 = warp * pw * 16;  // columns of O
+    const int np = max(0, min(pw, pairs - warp * pw));
+    float o[MT][NP][2][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int i = 0; i < NP; i++)
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) o[m][i][k][e] = 0.f;
+    const int lr = lane & 15, lc = (lane >> 4) * 8;   // ldmatrix x4: row, column offset (A operand; transposed B operand)
+    const int br = (lane & 7) + (lane >> 4) * 8, bc = ((lane >> 3) & 1) * 8;  // B operand from rows of keys: two n-tiles at once
+    int buf = 0;
+    for (int j = j0; j < j1; j += kSpKeys, buf ^= 1) {
+        cp_wait<0>();
+        __syncthreads();
+        if (j + kSpKeys < j1) load_tile(j + kSpKeys, buf ^ 1);
+        const bf16 *ct = cs + (size_t)buf * kSpKeys * pitch;
+        float s[MT][2][4];
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) s[m][k][e] = 0.f;
+#pragma unroll 4
+        for (int ks = ks0; ks < ks1; ks++) {
+            uint32_t b[4];
+            ldsm4(b, smem_addr(ct + (kg * 16 + br) * pitch + ks * 16 + bc));
+#pragma unroll
+            for (int m = 0; m < MT; m++) {
+                uint32_t a[4];
+                ldsm4(a, smem_addr(qs + (m * 16 + lr) * pitch + ks * 16 + lc));
+                mma16816(s[m][0], a, b[0], b[1]);
+                mma16816(s[m][1], a, b[2], b[3]);
+            }
+        }
+        const int g = lane >> 2, t = lane & 3;
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int k = 0; k < 2; k++) {
+                float *d = ss + ((size_t)rq * HM + m * 16 + g) * (kSpKeys + 2) + kg * 16 + k * 8 + 2 * t;
+                *reinterpret_cast<float2 *>(d) = make_float2(s[m][k][0], s[m][k][1]);
+                *reinterpret_cast<float2 *>(d + 8 * (kSpKeys + 2)) = make_float2(s[m][k][2], s[m][k][3]);
+            }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < HM / kSpWarps; i++) {
+            const int r = warp * (HM / kSpWarps) + i;
+            float v = 0.f;
+#pragma unroll
+            for (int k = 0; k < 4; k++) v += ss[((size_t)k * HM + r) * (kSpKeys + 2) + lane];
+            v = j + lane < j1 ? v * p.scale_log2 : -INFINITY;
+            float m = v;
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
+            const float mo = mrow[r];
+            m = fmaxf(m, mo);
+            const float e = exp2f(v - m);
+            float sum = e;
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+            ps[r * (kSpKeys + 8) + lane] = __float2bfloat16_rn(e);
+            __syncwarp();
+            if (lane == 0) {
+                const float f = exp2f(mo - m);
+                fac[r] = f;
+                lrow[r] = lrow[r] * f + sum;
+                mrow[r] = m;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+            const float f0 = fac[m * 16 + g], f1 = fac[m * 16 + g + 8];
+#pragma unroll
+            for (int i = 0; i < NP; i++)
+#pragma unroll
+                for (int k = 0; k < 2; k++) {
+                    o[m][i][k][0] *= f0;
+                    o[m][i][k][1] *= f0;
+                    o[m][i][k][2] *= f1;
+                    o[m][i][k][3] *= f1;
+                }
+        }
+#pragma unroll
+        for (int kk = 0; kk < kSpKeys / 16; kk++) {
+            uint32_t a[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; m++) ldsm4(a[m], smem_addr(ps + (m * 16 + lr) * (kSpKeys + 8) + kk * 16 + lc));
+#pragma unroll
+            for (int i = 0; i < NP; i++) {
+                if (i < np) {
+                    uint32_t b[4];
+                    ldsm4_trans(b, smem_addr(ct + (kk * 16 + lr) * pitch + c0 + i * 16 + lc));
+#pragma unroll
+                    for (int m = 0; m < MT; m++) {
+                        mma16816(o[m][i][0], a[m], b[0], b[1]);
+                        mma16816(o[m][i][1], a[m], b[2], b[3]);
+                    }
+                }
+            }
+        }
+    }
+    __syncthreads();
+    const int g = lane >> 2, t = lane & 3;
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int i = 0; i < NP; i++)
+            if (i < np)
+#pragma unroll
+                for (int k = 0; k < 2; k++) {
+                    const int col = c0 + i * 16 + k * 8 + 2 * t, ha = m * 16 + g, hb = ha + 8;
+                    if (ha < nh) *reinterpret_cast<float2 *>(p.part_o + (part + (size_t)ha * p.n_splits) * R + col) = make_float2(o[m][i][k][0], o[m][i][k][1]);
+                    if (hb < nh) *reinterpret_cast<float2 *>(p.part_o + (part + (size_t)hb * p.n_splits) * R + col) = make_float2(o[m][i][k][2], o[m][i][k][3]);
+                }
+    if (tid < nh) {
+        p.part_ml[(part + (size_t)tid * p.n_splits) * 2] = mrow[tid];
+        p.part_ml[(part + (size_t)tid * p.n_splits) * 2 + 1] = lrow[tid];
+    }
+}
+
+// ───────────────────────────── merge + value projection ───────────────────────────────────
+constexpr int kMergeThreads = 256, kMaxSplits = 64;
+struct MergeParams {
+    LatentMergeArgs a;
+    int rows_per;  // value rows of a block
+};
+__global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const MergeParams p) {
+    extern __shared__ __align__(16) float ol[];  // [rank]
+    __shared__ float wsp[kMaxSplits];
+    const LatentMergeArgs &a = p.a;
+    const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t part = ((size_t)row * a.heads + h) * a.n_splits;
+    if (warp == 0) {
+        float m0 = lane < a.n_splits ? a.part_ml[(part + lane) * 2] : -INFINITY, m1 = lane + 32 < a.n_splits ? a.part_ml[(part + lane + 32) * 2] : -INFINITY;
+        float l0 = lane < a.n_splits ? a.part_ml[(part + lane) * 2 + 1] : 0.f, l1 = lane + 32 < a.n_splits ? a.part_ml[(part + lane + 32) * 2 + 1] : 0.f;
+        float m = fmaxf(m0, m1);
+#pragma unroll
+        for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
+        const float f0 = exp2f(m0 - m), f1 = exp2f(m1 - m);
+        float l = l0 * f0 + l1 * f1;
+#pragma unroll
+        for (int d = 16; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+        wsp[lane] = f0 / l;
+        wsp[lane + 32] = f1 / l;
+    }
+    __syncthreads();
+    for (int c = tid * 4; c < a.rank; c += kMergeThreads * 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s = 0; s < a.n_splits; s++) {
+            const float w = wsp[s];
+            if (w == 0.f) continue;  // an empty split has written no rows
+            const float4 x = load4(a.part_o + (part + s) * a.rank + c);
+            v.x = fmaf(w, x.x, v.x);
+            v.y = fmaf(w, x.y, v.y);
+            v.z = fmaf(w, x.z, v.z);
+            v.w = fmaf(w, x.w, v.w);
+        }
+        store4(ol + c, v);
+    }
+    __syncthreads();
+    const float gate = sigmoid_f32(a.gate[(size_t)row * a.ld_gate + h]);
+    const int v0 = blockIdx.z * p.rows_per, v1 = min(a.vdim, v0 + p.rows_per);
+    for (int v = v0 + warp; v < v1; v += kMergeThreads / 32) {
+        const bf16 *w = static_cast<const bf16 *>(a.w_uv) + ((size_t)h * a.vdim + v) * a.rank;
+        float acc = 0.f;
+        for (int c = lane * 4; c < a.rank; c += 128) {
+            const float4 x = load4(w + c), y = load4(ol + c);
+            acc = fmaf(x.x, y.x, acc);
+            acc = fmaf(x.y, y.y, acc);
+            acc = fmaf(x.z, y.z, acc);
+            acc = fmaf(x.w, y.w, acc);
+        }
+#pragma unroll
+        for (int d = 16; d > 0; d >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, d);
+        if (lane == 0) static_cast<bf16 *>(a.out)[(size_t)row * a.heads * a.vdim + (size_t)h * a.vdim + v] = __float2bfloat16_rn(acc * gate);
+    }
+}
+
+// ───────────────────────────── prompts: causal flash attention ────────────────────────────
+// 128 query rows of one head per CTA, four warps of MT 16-row tiles; 64 keys per step, keys and values double-buffered.
+constexpr int kFlKeys = 64, kFlThreads = 128;
+struct FlashParams {
+    FlashArgs a;
+    float scale_log2;
+};
+template <int D, int MT>  // D: most dimensions per head; MT: 16-row tiles per warp
+__global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_kernel(const FlashParams p) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    constexpr int BR = 64 * MT, NK = D / 16, NV = D / 16;
+    const FlashArgs &a = p.a;
+    const int dp = a.dim, vp = a.vdim, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
+    bf16 *qs = reinterpret_cast<bf16 *>(sm);
+    bf16 *ks = qs + BR * kp;                 // [2][64][kp]
+    bf16 *vs = ks + 2 * kFlKeys * kp;        // [2][64][vpitch]
+    const int h = blockIdx.y, r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * BR;  // long rows first
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const bf16 *q = static_cast<const bf16 *>(a.q) + (size_t)h * dp;
+    const bf16 *kv = static_cast<const bf16 *>(a.kv);
+    const int ldq = a.heads * dp, rows = min(BR, a.n - r0), len = a.pos0 + r0 + rows;  // keys any row of the tile sees
+    const int kc = dp >> 3, vc = vp >> 3;
+    auto load_kv = [&](int j, int buf) {
+        for (int i = tid; i < kFlKeys * kc; i += kFlThreads) {
+            const int r = i / kc, ch = i - r * kc;
+            const bool ok = j + r < len;
+            cp16(smem_addr(ks + ((size_t)buf * kFlKeys + r) * kp + ch * 8), kv + (size_t)(ok ? j + r : 0) * a.ldkv + h * dp + ch * 8, ok);
+        }
+        for (int i = tid; i < kFlKeys * vc; i += kFlThreads) {
+            const int r = i / vc, ch = i - r * vc;
+            const bool ok = j + r < len;
+            cp16(smem_addr(vs + ((size_t)buf * kFlKeys + r) * vpitch + ch * 8), kv + (size_t)(ok ? j + r : 0) * a.ldkv + a.heads * dp + h * vp + ch * 8, ok);
+        }
+        cp_commit();
+    };
+    for (int i = tid; i < BR * kc; i += kFlThreads) {
+        const int r = i / kc, ch = i - r * kc;
+        const bool ok = r < rows;
+        cp16(smem_addr(qs + r * kp + ch * 8), q + (size_t)(ok ? r0 + r : r0) * ldq + ch * 8, ok);
+    }
+    load_kv(0, 0);
+    const int lr = lane & 15, lc = (lane >> 4) * 8, br = (lane & 7) + (lane >> 4) * 8, bc = ((lane >> 3) & 1) * 8;
+    const int g = lane >> 2, t = lane & 3, wrow = warp * 16 * MT;
+    float o[MT][NV][2][4], mx[MT][2], ls[MT][2];
+#pragma unroll
+    for (int m = 0; m < MT; m++) {
+        mx[m][0] = mx[m][1] = -INFINITY;
+        ls[m][0] = ls[m][1] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) o[m][i][k][e] = 0.f;
+    }
+    int buf = 0;
+    for (int j = 0; j < len; j += kFlKeys, buf ^= 1) {
+        cp_wait<0>();
+        __syncthreads();
+        if (j + kFlKeys < len) load_kv(j + kFlKeys, buf ^ 1);
+        if (j > a.pos0 + r0 + wrow + 16 * MT - 1) continue;  // every key of the tile lies behind this warp's rows
+        const bf16 *kt = ks + (size_t)buf * kFlKeys * kp, *vt = vs + (size_t)buf * kFlKeys * vpitch;
+        float s[MT][kFlKeys / 8][4];
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int i = 0; i < kFlKeys / 8; i++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) s[m][i][e] = 0.f;
+#pragma unroll
+        for (int k = 0; k < NK; k++) {
+            if (k < nk) {
+                uint32_t qa[MT][4];
+#pragma unroll
+                for (int m = 0; m < MT; m++) ldsm4(qa[m], smem_addr(qs + (wrow + m * 16 + lr) * kp + k * 16 + lc));
+#pragma unroll
+                for (int i = 0; i < kFlKeys / 16; i++) {
+                    uint32_t b[4];
+                    ldsm4(b, smem_addr(kt + (i * 16 + br) * kp + k * 16 + bc));
+#pragma unroll
+                    for (int m = 0; m < MT; m++) {
+                        mma16816(s[m][2 * i], qa[m], b[0], b[1]);
+                        mma16816(s[m][2 * i + 1], qa[m], b[2], b[3]);
+                    }
+                }
+            }
+        }
+        uint32_t pa[MT][kFlKeys / 16][4];
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+#pragma unroll
+            for (int e2 = 0; e2 < 2; e2++) {  // rows g and g + 8
+                const int pos = a.pos0 + r0 + wrow + m * 16 + g + e2 * 8;
+                float mv = mx[m][e2];
+                if (j + kFlKeys - 1 > pos) {
+#pragma unroll
+                    for (int i = 0; i < kFlKeys / 8; i++)
+#pragma unroll
+                        for (int e = 0; e < 2; e++)
+                            if (j + i * 8 + 2 * t + e > pos) s[m][i][e2 * 2 + e] = -INFINITY;
+                }
+#pragma unroll
+                for (int i = 0; i < kFlKeys / 8; i++) mv = fmaxf(mv, fmaxf(s[m][i][e2 * 2], s[m][i][e2 * 2 + 1]));
+                mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 1));
+                mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 2));
+                const float base = mv == -INFINITY ? 0.f : mv * p.scale_log2;
+                const float f = exp2f(mx[m][e2] * p.scale_log2 - base);
+                mx[m][e2] = mv;
+                float sum = 0.f;
+#pragma unroll
+                for (int i = 0; i < kFlKeys / 8; i++)
+#pragma unroll
+                    for (int e = 0; e < 2; e++) {
+                        const float v = exp2f(fmaf(s[m][i][e2 * 2 + e], p.scale_log2, -base));
+                        s[m][i][e2 * 2 + e] = v;
+                        sum += v;
+                    }
+                ls[m][e2] = ls[m][e2] * f + sum;
+#pragma unroll
+                for (int i = 0; i < NV; i++)
+#pragma unroll
+                    for (int k = 0; k < 2; k++) {
+                        o[m][i][k][e2 * 2] *= f;
+                        o[m][i][k][e2 * 2 + 1] *= f;
+                    }
+            }
+#pragma unroll
+            for (int i = 0; i < kFlKeys / 16; i++) {
+                pa[m][i][0] = pack_bf16(s[m][2 * i][0], s[m][2 * i][1]);
+                pa[m][i][1] = pack_bf16(s[m][2 * i][2], s[m][2 * i][3]);
+                pa[m][i][2] = pack_bf16(s[m][2 * i + 1][0], s[m][2 * i + 1][1]);
+                pa[m][i][3] = pack_bf16(s[m][2 * i + 1][2], s[m][2 * i + 1][3]);
+            }
+        }
+#pragma unroll
+        for (int kk = 0; kk < kFlKeys / 16; kk++)
+#pragma unroll
+            for (int i = 0; i < NV; i++) {
+                if (i < nv) {
+                    uint32_t b[4];
+                    ldsm4_trans(b, smem_addr(vt + (kk * 16 + lr) * vpitch + i * 16 + lc));
+#pragma unroll
+                    for (int m = 0; m < MT; m++) {
+                        mma16816(o[m][i][0], pa[m][kk], b[0], b[1]);
+                        mma16816(o[m][i][1], pa[m][kk], b[2], b[3]);
+                    }
+                }
+            }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int e2 = 0; e2 < 2; e2++) {
+            float l = ls[m][e2];
+            l += __shfl_xor_sync(0xffffffffu, l, 1);
+            l += __shfl_xor_sync(0xffffffffu, l, 2);
+            const int r = wrow + m * 16 + g + e2 * 8;
+            if (r >= rows) continue;
+            float f = 1.f / l;
+            if (a.gate) f *= sigmoid_f32(a.gate[(size_t)(r0 + r) * a.ld_gate + h]);
+            bf16 *out = static_cast<bf16 *>(a.out) + (size_t)(r0 + r) * a.heads * vp + h * vp;
+#pragma unroll
+            for (int i = 0; i < NV; i++)
+                if (i < nv)
+#pragma unroll
+                    for (int k = 0; k < 2; k++)
+                        *reinterpret_cast<uint32_t *>(out + i * 16 + k * 8 + 2 * t) = pack_bf16(o[m][i][k][e2 * 2] * f, o[m][i][k][e2 * 2 + 1] * f);
+        }
+}
+
+__global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t *plane, const int32_t *table, int max_pages, const int32_t *slot_of, int len,
+                                                            int row_bytes, uint8_t *out) {
+    const int per = row_bytes >> 4;
+    const int32_t *row = table + (size_t)*slot_of * max_pages;
+    for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < (size_t)len * per; i += (size_t)gridDim.x * 256) {
+        const int j = (int)(i / per), ch = (int)(i - (size_t)j * per);
+        const uint4 v = *reinterpret_cast<const uint4 *>(plane + ((size_t)row[j >> 4] * kPageTokens + (j & (kPageTokens - 1))) * row_bytes + ch * 16);
+        *reinterpret_cast<uint4 *>(out + (size_t)j * row_bytes + ch * 16) = v;
+    }
+}
+
+// ───────────────────────────── launches ───────────────────────────────────────────────────
+static int head_groups(int heads) { return heads <= 16 ? 1 : (heads + 31) / 32; }
+
+int latent_pick_splits(const juno_ctx *c, int n, int heads, int len_bound) {
+    const int want = std::max(1, 2 * c->sm_count / std::max(1, n * head_groups(heads)));
+    const int most = std::max(1, (len_bound + 2 * kSpKeys - 1) / (2 * kSpKeys));  // at least 64 positions each
+    return std::max(1, std::min(std::min(want, most), kMaxSplits));
+}
+size_t latent_part_floats(const juno_ctx *c, int n, int heads, int rank) {
+    const int groups = head_groups(heads);
+    return (size_t)std::min<long long>((long long)n * groups * kMaxSplits, 2ll * c->sm_count + (long long)n * groups) * (heads <= 16 ? 16 : 32) * (rank + 2);
+}
+
+template <int MT, int NP>
+static int split_launch(juno_ctx *c, const SplitParams &p, int n, cudaStream_t st) {
+    constexpr int HM = 16 * MT;
+    const size_t smem = (size_t)(HM + 2 * kSpKeys) * (p.rank + 8) * 2 + (size_t)HM * (kSpKeys + 8) * 2 + (size_t)4 * HM * (kSpKeys + 2) * 4 + (size_t)3 * HM * 4;
+    auto kernel = latent_split_kernel<MT, NP>;
+    static std::mutex mu;
+    static size_t have[16] = {0};
+    {
+        std::lock_guard<std::mutex> lk(mu);
+        if (smem > have[c->device & 15]) {
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            have[c->device & 15] = smem;
+        }
+    }
+    JUNO_CUDA_TRY(launch_pdl(kernel, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
+    c->kernel_launches++;
+    return JUNO_OK;
+}
+
+int launch_latent_attn_split(juno_ctx *c, const LatentSplitArgs &a, cudaStream_t st) {
+    JUNO_REQUIRE(a.rows.n > 0 && a.heads > 0 && a.rank % 16 == 0 && a.rank <= kLatentSplitMaxRank && a.pool->latent && a.pool->dtype == 2 &&
+                     a.pool->row_width[a.layer] == a.rank && a.n_splits >= 1 && a.n_splits <= kMaxSplits,
+                 "latent attention (splits): bad arguments");
+    SplitParams p;
+    p.plane = reinterpret_cast<const bf16 *>(static_cast<const uint8_t *>(a.pool->k) + a.pool->row_off[a.layer] * 2);
+    p.table = a.pool->d_table;
+    p.positions = a.rows.positions;
+    p.slots = a.rows.slots;
+    p.max_pages = a.pool->max_pages_per_seq;
+    p.heads = a.heads;
+    p.rank = a.rank;
+    p.n_splits = a.n_splits;
+    p.scale_log2 = a.scale * kLog2e;
+    p.q = static_cast<const bf16 *>(a.q_lat);
+    p.part_o = a.part_o;
+    p.part_ml = a.part_ml;
+    ProfScope prof(c, st, PROF_ATTN, 0);
+    const int n = a.rows.n, pw = ((a.rank >> 4) + kSpWarps - 1) / kSpWarps;
+    if (a.heads <= 16) return pw <= 1 ? split_launch<1, 1>(c, p, n, st) : pw <= 4 ? split_launch<1, 4>(c, p, n, st) : split_launch<1, 8>(c, p, n, st);
+    return pw <= 1 ? split_launch<2, 1>(c, p, n, st) : pw <= 4 ? split_launch<2, 4>(c, p, n, st) : split_launch<2, 8>(c, p, n, st);
+}
+
+int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st) {
+    JUNO_REQUIRE(a.n > 0 && a.heads > 0 && a.rank % 16 == 0 && a.rank <= kLatentSplitMaxRank && a.n_splits >= 1 && a.n_splits <= kMaxSplits, "latent merge: bad arguments");
+    MergeParams p;
+    p.a = a;
+    int parts = std::max(1, std::min((a.vdim + 15) / 16, (c->sm_count + a.n * a.heads - 1) / (a.n * a.heads)));
+    p.rows_per = (a.vdim + parts - 1) / parts;
+    parts = (a.vdim + p.rows_per - 1) / p.rows_per;
+    ProfScope prof(c, st, PROF_ATTN, 0);
+    JUNO_CUDA_TRY(launch_pdl(latent_merge_kernel, dim3((unsigned)a.heads, (unsigned)a.n, (unsigned)parts), dim3(kMergeThreads), (size_t)a.rank * 4, st, p));
+    c->kernel_launches++;
+    return JUNO_OK;
+}
+
+template <int D, int MT>
+static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
+    constexpr int BR = 64 * MT;
+    const size_t smem = ((size_t)(BR + 2 * kFlKeys) * (p.a.dim + 8) + (size_t)2 * kFlKeys * (p.a.vdim + 8)) * 2;
+    static std::mutex mu;
+    static size_t have[16] = {0};
+    {
+        std::lock_guard<std::mutex> lk(mu);
+        if (smem > have[c->device & 15]) {
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(flash_prefill_kernel<D, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            have[c->device & 15] = smem;
+        }
+    }
+    flash_prefill_kernel<D, MT><<<dim3((unsigned)((p.a.n + BR - 1) / BR), (unsigned)p.a.heads), kFlThreads, smem, st>>>(p);
+    JUNO_CUDA_TRY(cudaGetLastError());
+    c->kernel_launches++;
+    return JUNO_OK;
+}
+
+int launch_flash_prefill(juno_ctx *c, const FlashArgs &a, cudaStream_t st) {
+    JUNO_REQUIRE(a.n > 0 && a.pos0 >= 0 && a.heads > 0 && a.dim % 16 == 0 && a.vdim % 16 == 0 && a.dim <= kFlashMaxDim && a.vdim <= kFlashMaxDim && a.ldkv % 8 == 0,
+                 "prompt attention: bad arguments (dim %d, vdim %d)", a.dim, a.vdim);
+    FlashParams p;
+    p.a = a;
+    p.scale_log2 = a.scale * kLog2e;
+    const double pairs = (double)a.n * a.pos0 + (double)a.n * (a.n + 1) / 2;
+    ProfScope prof(c, st, PROF_ATTN, pairs * 2);
+    const int d = std::max(a.dim, a.vdim);
+    if (d <= 64) return flash_launch<64, 2>(c, p, st);
+    if (d <= 128) return flash_launch<128, 2>(c, p, st);
+    return flash_launch<256, 1>(c, p, st);
+}
+
+int launch_latent_gather(juno_ctx *c, const juno_kvpool *pool, int layer, const int32_t *slot_of, int len, void *out, cudaStream_t st) {
+    JUNO_REQUIRE(pool->latent && len > 0, "latent gather: bad arguments");
+    const int row_bytes = pool->row_width[layer] * pool->elem_bytes;
+    const size_t n = (size_t)len * (row_bytes >> 4);
+    ProfScope prof(c, st, PROF_ROWOPS, 2.0 * len * row_bytes);
+    latent_gather_kernel<<<(unsigned)std::min<size_t>((n + 255) / 256, 4 * (size_t)c->sm_count), 256, 0, st>>>(
+        static_cast<const uint8_t *>(pool->k) + pool->row_off[layer] * pool->elem_bytes, pool->d_table, pool->max_pages_per_seq, slot_of, len, row_bytes,
+        static_cast<uint8_t *>(out));
+    JUNO_CUDA_TRY(cudaGetLastError());
+    c->kernel_launches++;
+    return JUNO_OK;
+}
+
+}  // namespace juno

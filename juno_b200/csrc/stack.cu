@@ -95,13 +95,21 @@ int stack_upload_f32(juno_ctx *c, StackNet *net, const std::vector<float> &v, fl
     return JUNO_OK;
 }
 
+// A portion of a prompt with at most this many positions attends with absorbed queries, like a decode step: expanding keys and
+// values from the whole context would cost more than it saves.
+constexpr int kAbsorbRows = 48;
+static bool flash_fits(const LatentMixerSpec &m) { return m.dp() <= kFlashMaxDim && m.vp() <= kFlashMaxDim; }
+
 // ───────────────────────────── buffers ────────────────────────────────────────────────────
 int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int logit_rows) {
     const StackSpec &s = net->spec;
     const size_t es = dt_bytes(net->dt);
     const int cap = net->cap = std::max(max_batch, max_rows);
-    net->lat_cap = cap;
     net->logit_cap = logit_rows;
+    // absorbed queries are kept for few rows only, unless some layer has to take the general kernel
+    net->lat_cap = net->dt == DT_BF16 ? std::min(cap, std::max(max_batch, kAbsorbRows)) : cap;
+    for (const StackLayerSpec &L : s.layers)
+        if (!flash_fits(L.mix) || L.mix.rp() > kLatentSplitMaxRank) net->lat_cap = cap;
     const int wp = s.wp();
     int ff = 16;
     for (const StackLayerSpec &L : s.layers) {
@@ -114,6 +122,11 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
         ff = std::max(ff, pad16(L.ff));
     }
     net->ldact = ff;
+    if (net->dt == DT_BF16) {
+        for (const StackLayerSpec &L : s.layers)
+            for (int n = 1; n <= net->lat_cap; n++) net->part_floats = std::max(net->part_floats, latent_part_floats(c, n, L.mix.heads, L.mix.rp()));
+        JUNO_TRY(net_alloc(net, (void **)&net->part_o, net->part_floats * 4));
+    }
     const struct { void **p; size_t bytes; } bufs[] = {
         {(void **)&net->x, (size_t)cap * wp * 4},
         {(void **)&net->u, (size_t)cap * net->ldu * 4},
@@ -142,19 +155,91 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
 void stack_free(StackNet *net) {
     if (!net) return;
     for (void *p : net->owned) cudaFree(p);
+    if (net->ctx_lat) cudaFree(net->ctx_lat);
+    if (net->ctx_kv) cudaFree(net->ctx_kv);
     delete net;
 }
 
 const float *stack_residual(const StackNet *net) { return net->last_x ? net->x2 : net->x; }
 
 int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bound) {
-    (void)c, (void)net, (void)n, (void)len_bound;
-    return 1;
+    if (net->dt != DT_BF16) return 1;
+    int heads = 1;
+    for (const StackLayerSpec &L : net->spec.layers) heads = std::max(heads, L.mix.heads);
+    return latent_pick_splits(c, n, heads, len_bound);
+}
+
+// ───────────────────────────── attention of one layer ─────────────────────────────────────
+// q -> att, the head gates applied.  Few rows: the queries are taken into the latent space (q_lat[h] = W_uk[h]^T q[h]) and
+// attend the latent pages themselves.  Many rows of one sequence: keys and values are expanded once for the pass.
+static int attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, const LatentMixerSpec &m, const juno_kvpool *pool, int layer,
+                     const RowSet &rows, int n_splits, int len_bound, cudaStream_t st) {
+    const int n = rows.n, dt = net->dt, H = m.heads, rp = m.rp(), dp = m.dp(), vp = m.vp();
+    unsigned *err = c->gemv_scratch.qerr;
+    const float *gate = net->u + m.gate_col();
+    GemmArgs g;
+    g.M = n;
+    if (dt == DT_BF16 && rows.one_seq && n > kAbsorbRows && flash_fits(m)) {
+        JUNO_TRY(ensure_device(&net->ctx_lat, &net->ctx_lat_bytes, (size_t)len_bound * rp * 2));
+        JUNO_TRY(ensure_device(&net->ctx_kv, &net->ctx_kv_bytes, (size_t)len_bound * H * (dp + vp) * 2));
+        JUNO_TRY(launch_latent_gather(c, pool, layer, rows.slots, len_bound, net->ctx_lat, st));
+        g.a = net->ctx_lat;
+        g.lda = rp;
+        g.w = L.ukv.w;
+        g.ldw = rp;
+        g.M = len_bound;
+        g.N = H * (dp + vp);
+        g.K = rp;
+        g.out = net->ctx_kv;
+        g.ldo = H * (dp + vp);
+        JUNO_TRY(launch_gemm_rows(c, dt, g, err, st));
+        FlashArgs f{n, len_bound - n, H, dp, vp, m.scale, net->q, net->ctx_kv, H * (dp + vp), gate, net->ldu, net->att};
+        return launch_flash_prefill(c, f, st);
+    }
+    JUNO_REQUIRE(n <= net->lat_cap, "a pass of %d rows exceeds the latent buffers (%d)", n, net->lat_cap);
+    g.a = net->q;
+    g.lda = H * dp;
+    g.w = L.ukt.w;
+    g.ldw = dp;
+    g.N = rp;
+    g.K = dp;
+    g.out = net->qlat;
+    g.ldo = H * rp;
+    g.groups = H;
+    g.a_step = dp;
+    g.w_step = rp;
+    g.o_step = rp;
+    JUNO_TRY(launch_gemm_rows(c, dt, g, err, st));
+    const uint8_t *w_uv = static_cast<const uint8_t *>(L.ukv.w) + (size_t)H * dp * rp * dt_bytes(dt);
+    if (dt == DT_BF16 && rp <= kLatentSplitMaxRank) {
+        const size_t ml = (size_t)n * H * n_splits * rp;
+        JUNO_REQUIRE(ml + (size_t)n * H * n_splits * 2 <= net->part_floats, "%d context splits of %d rows exceed the buffer", n_splits, n);
+        LatentSplitArgs sp{pool, layer, rows, H, rp, n_splits, m.scale, net->qlat, net->part_o, net->part_o + ml};
+        JUNO_TRY(launch_latent_attn_split(c, sp, st));
+        LatentMergeArgs mg{n, H, rp, vp, n_splits, net->part_o, net->part_o + ml, w_uv, gate, net->ldu, net->att};
+        return launch_latent_merge(c, mg, st);
+    }
+    LatentAttnArgs at{pool, layer, rows, H, rp, m.scale, net->qlat, net->olat};
+    JUNO_TRY(launch_latent_attn_simt(c, dt, at, st));
+    g.a = net->olat;
+    g.lda = H * rp;
+    g.w = w_uv;
+    g.ldw = rp;
+    g.N = vp;
+    g.K = rp;
+    g.out = net->att;
+    g.ldo = H * vp;
+    g.epi = GE_GROUP_GATE;
+    g.aux = gate;
+    g.ldaux = net->ldu;
+    g.a_step = rp;
+    g.w_step = vp;
+    g.o_step = vp;
+    return launch_gemm_rows(c, dt, g, err, st);
 }
 
 // ───────────────────────────── a pass over many rows ──────────────────────────────────────
 int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, cudaStream_t st) {
-    (void)n_splits, (void)len_bound;
     const StackSpec &s = net->spec;
     const int n = rows.n, wp = s.wp(), dt = net->dt, n_layers = (int)s.layers.size();
     unsigned *err = c->gemv_scratch.qerr;
@@ -208,41 +293,7 @@ int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
         LatentNormArgs ln{net->u, net->ldu, m.q_rank, m.kv_col(), m.kv_rank, L.dq_norm, L.dkv_norm, s.eps, net->cq, m.qp(), pool, l};
         JUNO_TRY(launch_latent_norm(c, dt, ln, rows, st));
         JUNO_TRY(product(net->cq, m.qp(), L.uq, net->q, m.heads * m.dp(), GE_OP));
-        {
-            GemmArgs g;  // q_lat[h] = W_uk[h]^T q[h]
-            g.a = net->q;
-            g.lda = m.heads * m.dp();
-            g.w = L.ukt.w;
-            g.ldw = L.ukt.cols;
-            g.M = n;
-            g.N = m.rp();
-            g.K = m.dp();
-            g.out = net->qlat;
-            g.ldo = m.heads * m.rp();
-            g.groups = m.heads;
-            g.a_step = m.dp();
-            g.w_step = m.rp();
-            g.o_step = m.rp();
-            JUNO_TRY(launch_gemm_rows(c, dt, g, err, st));
-            LatentAttnArgs at{pool, l, rows, m.heads, m.rp(), m.scale, net->qlat, net->olat};
-            JUNO_TRY(launch_latent_attn_simt(c, dt, at, st));
-            // out[h] = W_uv[h] o_lat[h] * sigmoid(gate[h])
-            g.a = net->olat;
-            g.lda = m.heads * m.rp();
-            g.w = static_cast<const uint8_t *>(L.ukv.w) + (size_t)m.heads * m.dp() * m.rp() * dt_bytes(dt);
-            g.ldw = m.rp();
-            g.N = m.vp();
-            g.K = m.rp();
-            g.out = net->att;
-            g.ldo = m.heads * m.vp();
-            g.epi = GE_GROUP_GATE;
-            g.aux = net->u + m.gate_col();
-            g.ldaux = net->ldu;
-            g.a_step = m.rp();
-            g.w_step = m.vp();
-            g.o_step = m.vp();
-            JUNO_TRY(launch_gemm_rows(c, dt, g, err, st));
-        }
+        JUNO_TRY(attention(c, net, L, m, pool, l, rows, n_splits, len_bound, st));
         JUNO_TRY(product(net->att, m.heads * m.vp(), L.o, net->z, wp, GE_MUL, nullptr, net->gate));
         const bool mlp = s.layers[l].ff > 0;
         JUNO_TRY(residual(net->z, L.norm1b, mlp || !last, mlp ? L.norm2 : next_norm1));

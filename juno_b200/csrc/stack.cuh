@@ -72,6 +72,10 @@ struct StackNet {
     void *h = nullptr, *hc = nullptr, *gate = nullptr, *z = nullptr, *cq = nullptr, *q = nullptr, *qlat = nullptr, *olat = nullptr,
          *att = nullptr, *act = nullptr, *fin = nullptr;
     int ldu = 0, ldcq = 0, ldq = 0, ldlat = 0, ldatt = 0, ldact = 0;
+    float *part_o = nullptr;  // partial results of the attention's context splits
+    size_t part_floats = 0;
+    void *ctx_lat = nullptr, *ctx_kv = nullptr;   // a prompt pass: the sequence's latents, and keys and values expanded from them
+    size_t ctx_lat_bytes = 0, ctx_kv_bytes = 0;
     int32_t *row_idx = nullptr;  // device list of rows whose logits are wanted
     double weight_bytes = 0;     // bytes a one-token step reads
     int last_x = 0;

@@ -47,6 +47,7 @@ int vosotar_spec(const Json &cfg, StackSpec *spec) {
         JUNO_TRY(get_int(m, "q_rank", wm.c_str(), 1, kMax, &L.mix.q_rank));
         JUNO_TRY(get_int(m, "kv_rank", wm.c_str(), 1, 2048, &L.mix.kv_rank));
         JUNO_TRY(get_float(m, "scale", wm.c_str(), &L.mix.scale));
+        JUNO_REQUIRE(L.mix.scale > 0.f, "config: %s.scale must be positive", wm.c_str());
         const Json *mlp = e.find("mlp");
         if (mlp && !mlp->is_null()) {
             const Json *kind = mlp->find("kind");
