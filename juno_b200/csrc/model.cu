@@ -1139,8 +1139,7 @@ static int enqueue_step(juno_model *m, int n, int n_splits, bool greedy_advance,
         rows.positions = d_pos;
         rows.slots = d_slot;
         rows.lens = d_len;
-        JUNO_TRY(stack_enqueue_layers(c, m->stack, m->pool, rows, n_splits, f.max_ctx, st));
-        JUNO_TRY(stack_enqueue_logits(c, m->stack, nullptr, n, m->logits_loc, st));
+        JUNO_TRY(stack_enqueue_step(c, m->stack, m->pool, rows, n_splits, f.max_ctx, m->logits_loc, st));
         return enqueue_pick(m, n, greedy_advance, want_logits, st);
     }
     if (m->tp_push) {
@@ -1500,6 +1499,7 @@ int juno_forward(juno_model *m, int32_t n, juno_seq *const *seqs, const int32_t 
     JUNO_TRY(step_sync(m));
     JUNO_TRY(step_check(m));
     for (int i = 0; i < n; i++) seqs[i]->len = std::max(seqs[i]->len, positions[i] + 1);
+    if (m->stack) stack_step_done(c, m->stack, n);
     m->last_n = n;
     return JUNO_OK;
 }
@@ -1552,6 +1552,7 @@ int juno_decode_greedy(juno_model *m, int32_t n, juno_seq *const *seqs, const in
     JUNO_TRY(step_check(m));
     c->d2h_bytes += (int64_t)steps * n * 4;
     for (int i = 0; i < n; i++) seqs[i]->len = std::max(seqs[i]->len, positions[i] + steps);
+    if (m->stack) stack_step_done(c, m->stack, n);
     m->last_n = n;
     return JUNO_OK;
 }

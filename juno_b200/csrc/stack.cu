@@ -1,5 +1,6 @@
 // Layer stacks with dense weights: loading helpers, buffers, and the pass over many rows (portions of prompts, large decode
 // batches, and every pass in 32-bit).
+#include "gemv_rows.cuh"
 #include "stack.cuh"
 
 #include <algorithm>
@@ -122,6 +123,12 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
         ff = std::max(ff, pad16(L.ff));
     }
     net->ldact = ff;
+    net->weight_bytes = (double)net->head.rows * net->head.cols * es;
+    for (size_t l = 0; l < s.layers.size(); l++) {
+        const StackLayerWeights &L = net->layers[(size_t)s.weights((int)l)];
+        for (const StackMat *m : {&L.down, &L.uq, &L.ukt, &L.o, &L.rg1, &L.rg2, &L.up, &L.mdown}) net->weight_bytes += (double)m->rows * m->cols * es;
+        net->weight_bytes += (double)s.layers[l].mix.heads * s.layers[l].mix.vp() * s.layers[l].mix.rp() * es;  // W_uv
+    }
     if (net->dt == DT_BF16) {
         for (const StackLayerSpec &L : s.layers)
             for (int n = 1; n <= net->lat_cap; n++) net->part_floats = std::max(net->part_floats, latent_part_floats(c, n, L.mix.heads, L.mix.rp()));
@@ -143,6 +150,9 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
         {&net->act, (size_t)cap * net->ldact * es},
         {&net->fin, (size_t)std::max(logit_rows, 1) * wp * es},
         {(void **)&net->row_idx, (size_t)cap * 4},
+        {(void **)&net->x2, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
+        {(void **)&net->dec_gate, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
+        {(void **)&net->dec_z, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
     };
     for (const auto &b : bufs) {
         JUNO_TRY(net_alloc(net, b.p, b.bytes));
@@ -158,6 +168,23 @@ void stack_free(StackNet *net) {
     if (net->ctx_lat) cudaFree(net->ctx_lat);
     if (net->ctx_kv) cudaFree(net->ctx_kv);
     delete net;
+}
+
+int stack_enqueue_step(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, float *logits, cudaStream_t st) {
+    if (stack_fused_ok(c, net, rows)) {
+        JUNO_TRY(stack_enqueue_decode(c, net, pool, rows, n_splits, st));
+        return stack_enqueue_decode_logits(c, net, rows.n, logits, st);
+    }
+    JUNO_TRY(stack_enqueue_layers(c, net, pool, rows, n_splits, len_bound, st));
+    return stack_enqueue_logits(c, net, nullptr, rows.n, logits, st);
+}
+
+void stack_step_done(const juno_ctx *c, StackNet *net, int n) {
+    RowSet rows;
+    rows.n = n;
+    net->last_x = 0;
+    if (!stack_fused_ok(c, net, rows)) return;
+    for (const StackLayerSpec &L : net->spec.layers) net->last_x ^= L.ff ? 0 : 1;  // one hand-over per sublayer
 }
 
 const float *stack_residual(const StackNet *net) { return net->last_x ? net->x2 : net->x; }
@@ -241,6 +268,7 @@ static int attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, con
 // ───────────────────────────── a pass over many rows ──────────────────────────────────────
 int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, cudaStream_t st) {
     const StackSpec &s = net->spec;
+    net->last_x = 0;
     const int n = rows.n, wp = s.wp(), dt = net->dt, n_layers = (int)s.layers.size();
     unsigned *err = c->gemv_scratch.qerr;
     JUNO_REQUIRE(n >= 1 && n <= net->cap, "a pass of %d rows exceeds the buffers (%d)", n, net->cap);

@@ -78,7 +78,11 @@ struct StackNet {
     size_t ctx_lat_bytes = 0, ctx_kv_bytes = 0;
     int32_t *row_idx = nullptr;  // device list of rows whose logits are wanted
     double weight_bytes = 0;     // bytes a one-token step reads
+    // fused decode step: residual rows x / x2 in turn (last_x: which holds the newest), sublayer result not yet added to them
+    float *dec_gate = nullptr, *dec_z = nullptr;
     int last_x = 0;
+    bool pending = false;
+    float pending_g = 0.f;
 };
 
 // ── loading ──
@@ -103,6 +107,14 @@ void stack_free(StackNet *net);
 int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, cudaStream_t st);
 // logits[i] = head . norm(x[row_idx[i]]) (row_idx null: row i), n rows
 int stack_enqueue_logits(juno_ctx *c, StackNet *net, const int32_t *row_idx, int n, float *logits, cudaStream_t st);
+// The same for a decode step of few sequences, on fused products (stack_decode.cu).
+bool stack_fused_ok(const juno_ctx *c, const StackNet *net, const RowSet &rows);
+int stack_enqueue_decode(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, cudaStream_t st);
+int stack_enqueue_decode_logits(juno_ctx *c, StackNet *net, int n, float *logits, cudaStream_t st);
+// One step of n sequences, logits included, on whichever of the two fits.
+int stack_enqueue_step(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, int len_bound, float *logits, cudaStream_t st);
+// A captured step has run: where its residual stream ended.
+void stack_step_done(const juno_ctx *c, StackNet *net, int n);
 const float *stack_residual(const StackNet *net);  // residual stream of the last pass, rows of wp() floats
 int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bound);
 
