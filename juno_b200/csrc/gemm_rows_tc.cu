@@ -83,6 +83,8 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
 // 32 columns of one output row.  nv = columns that exist (0..32).
 template <int EPI>
 __device__ __forceinline__ void store_row(const GemmArgs &g, int z, int m, int n, int nv, const uint32_t (&r)[32]) {
@@ -101,7 +103,7 @@ __device__ __forceinline__ void store_row(const GemmArgs &g, int z, int m, int n
         return;
     }
     float gate = 1.f;
-    if (EPI == GE_GROUP_GATE) gate = sigmoid_f32(static_cast<const float *>(g.aux)[(size_t)m * g.ldaux + z]);
+    if (EPI == GE_GROUP_GATE) gate = fast_sigmoid(static_cast<const float *>(g.aux)[(size_t)m * g.ldaux + z]);
     bf16 *out = static_cast<bf16 *>(g.out) + o;
     const bf16 *aux = EPI == GE_MUL ? static_cast<const bf16 *>(g.aux) + (size_t)m * g.ldaux + n : nullptr;
 #pragma unroll
@@ -110,7 +112,7 @@ __device__ __forceinline__ void store_row(const GemmArgs &g, int z, int m, int n
         float4 v = make_float4(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), __uint_as_float(r[j + 2]), __uint_as_float(r[j + 3]));
         if (EPI == GE_SIGMOID) {
             const float4 b = *reinterpret_cast<const float4 *>(g.bias + n + j);
-            v = make_float4(sigmoid_f32(v.x + b.x), sigmoid_f32(v.y + b.y), sigmoid_f32(v.z + b.z), sigmoid_f32(v.w + b.w));
+            v = make_float4(fast_sigmoid(v.x + b.x), fast_sigmoid(v.y + b.y), fast_sigmoid(v.z + b.z), fast_sigmoid(v.w + b.w));
         } else if (EPI == GE_RELU2) {
             v = make_float4(fmaxf(v.x, 0.f), fmaxf(v.y, 0.f), fmaxf(v.z, 0.f), fmaxf(v.w, 0.f));
             v = make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w);
@@ -306,9 +308,18 @@ int launch_gemm_rows_tc(juno_ctx *c, const GemmArgs &a, unsigned *err, cudaStrea
     p.err = err;
     p.m_tiles = (a.M + kBM - 1) / kBM;
     p.k_steps = (a.K + kBK - 1) / kBK;
-    // the widest tile that still gives every SM one, and is not wider than the matrix
-    int bn = 256;
-    while (bn > 32 && ((bn / 2 >= a.N) || (long long)p.m_tiles * ((a.N + bn - 1) / bn) * a.groups < c->sm_count)) bn /= 2;
+    // tile width: rounds of tiles over the SMs, each as long as its columns and a fixed share (operand A, start-up, epilogue)
+    int bn = 32;
+    double best = 1e30;
+    for (int w = 256; w >= 32; w /= 2) {
+        if (w > 32 && w / 2 >= a.N) continue;
+        const long long tiles = (long long)p.m_tiles * ((a.N + w - 1) / w) * a.groups;
+        const double cost = (double)((tiles + c->sm_count - 1) / c->sm_count) * (w + 40);
+        if (cost < best) {
+            best = cost;
+            bn = w;
+        }
+    }
     p.n_tiles = (a.N + bn - 1) / bn;
     p.n_work = p.m_tiles * p.n_tiles * a.groups;
     p.stages = std::min(kMaxStages, 192 * 1024 / ((kBM + bn) * kBK * 2));

@@ -31,14 +31,15 @@ struct LatentSplitArgs {
     float *part_o, *part_ml;
 };
 constexpr int kLatentSplitMaxRank = 1024;
-int latent_pick_splits(const juno_ctx *c, int n, int heads, int len_bound);
+int latent_pick_splits(const juno_ctx *c, int n, int heads, int rank, int len_bound);
 size_t latent_part_floats(const juno_ctx *c, int n, int heads, int rank);  // enough for any split count latent_pick_splits returns
 int launch_latent_attn_split(juno_ctx *c, const LatentSplitArgs &a, cudaStream_t st);
-// Merges the splits and applies the value projection and the head gate: out[h] = W_uv[h] o_lat[h] * sigmoid(gate[h]).
+// Merges the splits and applies the value projection and the head gate: out[h] = W_uv[h] o_lat[h] * sigmoid(gate[h]); without
+// w_uv the merged o_lat itself ([n][heads * rank]).
 struct LatentMergeArgs {
     int n, heads, rank, vdim, n_splits;  // rank, vdim padded
     const float *part_o, *part_ml;
-    const void *w_uv;    // [heads * vdim][rank] BF16
+    const void *w_uv;    // [heads * vdim][rank] BF16, or null
     const float *gate;   // [n][ld_gate]
     int ld_gate;
     void *out;           // [n][heads * vdim] BF16

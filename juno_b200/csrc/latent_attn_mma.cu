@@ -12,10 +12,11 @@ using bf16 = __nv_bfloat16;
 constexpr float kLog2e = 1.4426950408889634f;
 
 // ───────────────────────────── decode: splits of the context ──────────────────────────────
-// A CTA takes a group of 16 * MT heads of one row and a range of positions, 32 at a time.  Scores: warp (rank quarter, 16
-// positions) multiplies its part of q_lat with the tile, the four quarters are added in shared memory; online softmax by rows;
-// then each warp owns a range of latent columns of O += P C, reading the same tile transposed.
-constexpr int kSpKeys = 32, kSpThreads = 256, kSpWarps = 8;
+// A CTA (sixteen warps, one per SM) takes a group of 16 * MT heads of one row and a range of positions, KT at a time, the next
+// tile in flight.  Scores: warp (16 positions, part of the rank) multiplies its part of q_lat with the tile, the parts are added
+// in shared memory; online softmax by rows; then each warp owns a range of latent columns of O += P C, reading the same tile
+// transposed.
+constexpr int kSpThreads = 512, kSpWarps = 16;
 
 struct SplitParams {
     const bf16 *plane;
@@ -26,23 +27,35 @@ struct SplitParams {
     float *part_o, *part_ml;
 };
 
-template <int MT, int NP>  // NP: 16-column pairs of n-tiles a warp owns at most
-__global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_split_kernel(const SplitParams p) {
+__device__ __forceinline__ float ex2(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+
+template <int MT, int KT>
+constexpr size_t split_smem(int rank) {
+    return (size_t)(16 * MT + 2 * KT) * (rank + 8) * 2 + (size_t)16 * MT * (KT + 8) * 2 + (size_t)(kSpWarps * 16 / KT) * 16 * MT * (KT + 2) * 4 +
+           (size_t)3 * 16 * MT * 4;
+}
+
+template <int MT, int KT, int NP>  // NP: 16-column pairs of n-tiles a warp owns at most
+__global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const SplitParams p) {
     extern __shared__ __align__(16) uint8_t sm[];
-    constexpr int HM = 16 * MT;
+    constexpr int HM = 16 * MT, KG = KT / 16, RQ = kSpWarps / KG, SP = KT + 2;
     const int R = p.rank, pitch = R + 8;
     bf16 *qs = reinterpret_cast<bf16 *>(sm);          // [HM][pitch]
-    bf16 *cs = qs + HM * pitch;                       // [2][kSpKeys][pitch]
-    bf16 *ps = cs + 2 * kSpKeys * pitch;              // [HM][kSpKeys + 8]
-    float *ss = reinterpret_cast<float *>(ps + HM * (kSpKeys + 8));  // [4][HM][kSpKeys + 2]
-    float *fac = ss + 4 * HM * (kSpKeys + 2), *mrow = fac + HM, *lrow = mrow + HM;
+    bf16 *cs = qs + HM * pitch;                       // [2][KT][pitch]
+    bf16 *ps = cs + 2 * KT * pitch;                   // [HM][KT + 8]
+    float *ss = reinterpret_cast<float *>(ps + HM * (KT + 8));  // [RQ][HM][SP]
+    float *fac = ss + RQ * HM * SP, *mrow = fac + HM, *lrow = mrow + HM;
     const int split = blockIdx.x, h0 = blockIdx.y * HM, row = blockIdx.z, nh = min(HM, p.heads - h0);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_wait();
     pdl_launch_dependents();
     const int len = p.positions[row] + 1;
-    const int tiles = (len + kSpKeys - 1) / kSpKeys, per = (tiles + p.n_splits - 1) / p.n_splits;
-    const int j0 = split * per * kSpKeys, j1 = min(len, j0 + per * kSpKeys);
+    const int tiles = (len + KT - 1) / KT, per = (tiles + p.n_splits - 1) / p.n_splits;
+    const int j0 = split * per * KT, j1 = min(len, j0 + per * KT);
     const size_t part = ((size_t)row * p.heads + h0) * p.n_splits + split;  // + head * n_splits
     if (j0 >= j1) {
         if (tid < nh) {
@@ -53,22 +66,25 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
     }
     const int32_t *table = p.table + (size_t)p.slots[row] * p.max_pages;
     const int chunks = R >> 3;
+    // KT / 16 consecutive rows per warp: they lie in one page
+    constexpr int WR = KT / kSpWarps;
     auto load_tile = [&](int j, int buf) {
-        bf16 *dst = cs + (size_t)buf * kSpKeys * pitch;
-        for (int i = tid; i < kSpKeys * chunks; i += kSpThreads) {
-            const int r = i / chunks, ch = i - r * chunks;
-            const bool ok = j + r < j1;
-            const bf16 *src = latent_row(p.plane, table, R, ok ? j + r : j0) + ch * 8;
-            cp16(smem_addr(dst + r * pitch + ch * 8), src, ok);
+        const int r0 = warp * WR;
+        const bool any = j + r0 < j1;
+        const bf16 *src = any ? latent_row(p.plane, table, R, j + r0) : p.plane;
+        const uint32_t dst = smem_addr(cs + ((size_t)buf * KT + r0) * pitch);
+#pragma unroll
+        for (int i = 0; i < WR; i++) {
+            const bool ok = j + r0 + i < j1;
+            for (int ch = lane; ch < chunks; ch += 32) cp16(dst + (uint32_t)(i * pitch + ch * 8) * 2, ok ? src + (size_t)i * R + ch * 8 : p.plane, ok);
         }
         cp_commit();
     };
     {
         const bf16 *q = p.q + ((size_t)row * p.heads + h0) * R;
-        for (int i = tid; i < HM * chunks; i += kSpThreads) {
-            const int r = i / chunks, ch = i - r * chunks;
+        for (int r = warp; r < HM; r += kSpWarps) {
             const bool ok = r < nh;
-            cp16(smem_addr(qs + r * pitch + ch * 8), q + (ok ? (size_t)r * R + ch * 8 : 0), ok);
+            for (int ch = lane; ch < chunks; ch += 32) cp16(smem_addr(qs + r * pitch + ch * 8), ok ? q + (size_t)r * R + ch * 8 : q, ok);
         }
     }
     load_tile(j0, 0);
@@ -76,8 +92,8 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
         mrow[tid] = -INFINITY;
         lrow[tid] = 0.f;
     }
-    const int kg = warp & 1, rq = warp >> 1;                      // 16 positions, quarter of the rank
-    const int ksteps = R >> 4, ks0 = ksteps * rq / 4, ks1 = ksteps * (rq + 1) / 4;
+    const int kg = warp % KG, rq = warp / KG;                     // 16 positions, part of the rank
+    const int ksteps = R >> 4, ks0 = ksteps * rq / RQ, ks1 = ksteps * (rq + 1) / RQ;
     const int pairs = R >> 4, pw = (pairs + kSpWarps - 1) / kSpWarps, c0 = warp * pw * 16;  // columns of O
     const int np = max(0, min(pw, pairs - warp * pw));
     float o[MT][NP][2][4];
@@ -91,61 +107,74 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
                 for (int e = 0; e < 4; e++) o[m][i][k][e] = 0.f;
     const int lr = lane & 15, lc = (lane >> 4) * 8;   // ldmatrix x4: row, column offset (A operand; transposed B operand)
     const int br = (lane & 7) + (lane >> 4) * 8, bc = ((lane >> 3) & 1) * 8;  // B operand from rows of keys: two n-tiles at once
+    const int g = lane >> 2, t = lane & 3;
+    const uint32_t q_a = smem_addr(qs + lr * pitch + lc), p_a = smem_addr(ps + lr * (KT + 8) + lc);
     int buf = 0;
-    for (int j = j0; j < j1; j += kSpKeys, buf ^= 1) {
+    for (int j = j0; j < j1; j += KT, buf ^= 1) {
         cp_wait<0>();
         __syncthreads();
-        if (j + kSpKeys < j1) load_tile(j + kSpKeys, buf ^ 1);
-        const bf16 *ct = cs + (size_t)buf * kSpKeys * pitch;
-        float s[MT][2][4];
+        if (j + KT < j1) load_tile(j + KT, buf ^ 1);
+        const bf16 *ct = cs + (size_t)buf * KT * pitch;
+        {
+            float s[MT][2][4];
 #pragma unroll
-        for (int m = 0; m < MT; m++)
+            for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int k = 0; k < 2; k++)
+                for (int k = 0; k < 2; k++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) s[m][k][e] = 0.f;
+                    for (int e = 0; e < 4; e++) s[m][k][e] = 0.f;
+            const uint32_t k_a = smem_addr(ct + (kg * 16 + br) * pitch + bc);
 #pragma unroll 4
-        for (int ks = ks0; ks < ks1; ks++) {
-            uint32_t b[4];
-            ldsm4(b, smem_addr(ct + (kg * 16 + br) * pitch + ks * 16 + bc));
+            for (int ks = ks0; ks < ks1; ks++) {
+                uint32_t b[4];
+                ldsm4(b, k_a + ks * 32);
 #pragma unroll
-            for (int m = 0; m < MT; m++) {
-                uint32_t a[4];
-                ldsm4(a, smem_addr(qs + (m * 16 + lr) * pitch + ks * 16 + lc));
-                mma16816(s[m][0], a, b[0], b[1]);
-                mma16816(s[m][1], a, b[2], b[3]);
+                for (int m = 0; m < MT; m++) {
+                    uint32_t a[4];
+                    ldsm4(a, q_a + (uint32_t)(m * 16 * pitch + ks * 16) * 2);
+                    mma16816(s[m][0], a, b[0], b[1]);
+                    mma16816(s[m][1], a, b[2], b[3]);
+                }
             }
+#pragma unroll
+            for (int m = 0; m < MT; m++)
+#pragma unroll
+                for (int k = 0; k < 2; k++) {
+                    float *d = ss + (rq * HM + m * 16 + g) * SP + kg * 16 + k * 8 + 2 * t;
+                    *reinterpret_cast<float2 *>(d) = make_float2(s[m][k][0], s[m][k][1]);
+                    *reinterpret_cast<float2 *>(d + 8 * SP) = make_float2(s[m][k][2], s[m][k][3]);
+                }
         }
-        const int g = lane >> 2, t = lane & 3;
-#pragma unroll
-        for (int m = 0; m < MT; m++)
-#pragma unroll
-            for (int k = 0; k < 2; k++) {
-                float *d = ss + ((size_t)rq * HM + m * 16 + g) * (kSpKeys + 2) + kg * 16 + k * 8 + 2 * t;
-                *reinterpret_cast<float2 *>(d) = make_float2(s[m][k][0], s[m][k][1]);
-                *reinterpret_cast<float2 *>(d + 8 * (kSpKeys + 2)) = make_float2(s[m][k][2], s[m][k][3]);
-            }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < HM / kSpWarps; i++) {
             const int r = warp * (HM / kSpWarps) + i;
-            float v = 0.f;
+            float v[KT / 32];
+            float m = -INFINITY;
 #pragma unroll
-            for (int k = 0; k < 4; k++) v += ss[((size_t)k * HM + r) * (kSpKeys + 2) + lane];
-            v = j + lane < j1 ? v * p.scale_log2 : -INFINITY;
-            float m = v;
+            for (int x = 0; x < KT / 32; x++) {
+                v[x] = 0.f;
+#pragma unroll
+                for (int k = 0; k < RQ; k++) v[x] += ss[(k * HM + r) * SP + x * 32 + lane];
+                v[x] = j + x * 32 + lane < j1 ? v[x] * p.scale_log2 : -INFINITY;
+                m = fmaxf(m, v[x]);
+            }
 #pragma unroll
             for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
             const float mo = mrow[r];
             m = fmaxf(m, mo);
-            const float e = exp2f(v - m);
-            float sum = e;
+            float sum = 0.f;
+#pragma unroll
+            for (int x = 0; x < KT / 32; x++) {
+                const float e = ex2(v[x] - m);
+                sum += e;
+                ps[r * (KT + 8) + x * 32 + lane] = __float2bfloat16_rn(e);
+            }
 #pragma unroll
             for (int d = 16; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-            ps[r * (kSpKeys + 8) + lane] = __float2bfloat16_rn(e);
             __syncwarp();
             if (lane == 0) {
-                const float f = exp2f(mo - m);
+                const float f = ex2(mo - m);
                 fac[r] = f;
                 lrow[r] = lrow[r] * f + sum;
                 mrow[r] = m;
@@ -165,16 +194,17 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
                     o[m][i][k][3] *= f1;
                 }
         }
+        const uint32_t v_a = smem_addr(ct + lr * pitch + c0 + lc);
 #pragma unroll
-        for (int kk = 0; kk < kSpKeys / 16; kk++) {
+        for (int kk = 0; kk < KT / 16; kk++) {
             uint32_t a[MT][4];
 #pragma unroll
-            for (int m = 0; m < MT; m++) ldsm4(a[m], smem_addr(ps + (m * 16 + lr) * (kSpKeys + 8) + kk * 16 + lc));
+            for (int m = 0; m < MT; m++) ldsm4(a[m], p_a + (uint32_t)(m * 16 * (KT + 8) + kk * 16) * 2);
 #pragma unroll
             for (int i = 0; i < NP; i++) {
                 if (i < np) {
                     uint32_t b[4];
-                    ldsm4_trans(b, smem_addr(ct + (kk * 16 + lr) * pitch + c0 + i * 16 + lc));
+                    ldsm4_trans(b, v_a + (uint32_t)(kk * 16 * pitch + i * 16) * 2);
 #pragma unroll
                     for (int m = 0; m < MT; m++) {
                         mma16816(o[m][i][0], a[m], b[0], b[1]);
@@ -185,7 +215,6 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
         }
     }
     __syncthreads();
-    const int g = lane >> 2, t = lane & 3;
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
@@ -204,54 +233,82 @@ __global__ void __launch_bounds__(kSpThreads, (MT * NP <= 8) ? 2 : 1) latent_spl
 }
 
 // ───────────────────────────── merge + value projection ───────────────────────────────────
-constexpr int kMergeThreads = 256, kMaxSplits = 64;
+// One block per (head, row, share of the value rows).  The threads form groups that add up different splits of the averaged
+// latent; then every warp takes rows of W_uv.  Without w_uv the merged latent itself is the result (many rows: the value
+// projection is a matrix product then).
+constexpr int kMergeThreads = 512, kMaxSplits = 64;
 struct MergeParams {
     LatentMergeArgs a;
     int rows_per;  // value rows of a block
 };
 __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const MergeParams p) {
-    extern __shared__ __align__(16) float ol[];  // [rank]
+    __shared__ __align__(16) float acc_s[kMergeThreads * 4];
+    __shared__ __align__(16) float ol[kLatentSplitMaxRank];
     __shared__ float wsp[kMaxSplits];
     const LatentMergeArgs &a = p.a;
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int v0 = blockIdx.z * p.rows_per, v1 = min(a.vdim, v0 + p.rows_per);
+    const bf16 *wuv = static_cast<const bf16 *>(a.w_uv);
+    if (wuv)  // weights do not depend on the attention: on their way to L2 before it has finished
+        for (int i = tid; i < (v1 - v0) * a.rank / 64; i += kMergeThreads)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(wuv + ((size_t)h * a.vdim + v0) * a.rank + (size_t)i * 64));
     pdl_wait();
     pdl_launch_dependents();
     const size_t part = ((size_t)row * a.heads + h) * a.n_splits;
     if (warp == 0) {
-        float m0 = lane < a.n_splits ? a.part_ml[(part + lane) * 2] : -INFINITY, m1 = lane + 32 < a.n_splits ? a.part_ml[(part + lane + 32) * 2] : -INFINITY;
-        float l0 = lane < a.n_splits ? a.part_ml[(part + lane) * 2 + 1] : 0.f, l1 = lane + 32 < a.n_splits ? a.part_ml[(part + lane + 32) * 2 + 1] : 0.f;
-        float m = fmaxf(m0, m1);
+        const bool h0 = lane < a.n_splits, h1 = lane + 32 < a.n_splits;
+        const float2 z = make_float2(-INFINITY, 0.f), *ml = reinterpret_cast<const float2 *>(a.part_ml) + part;
+        const float2 e0 = h0 ? ml[lane] : z, e1 = h1 ? ml[lane + 32] : z;
+        float m = fmaxf(e0.x, e1.x);
 #pragma unroll
         for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
-        const float f0 = exp2f(m0 - m), f1 = exp2f(m1 - m);
-        float l = l0 * f0 + l1 * f1;
+        const float f0 = ex2(e0.x - m), f1 = ex2(e1.x - m);
+        float l = e0.y * f0 + e1.y * f1;
 #pragma unroll
         for (int d = 16; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
         wsp[lane] = f0 / l;
         wsp[lane + 32] = f1 / l;
     }
     __syncthreads();
-    for (int c = tid * 4; c < a.rank; c += kMergeThreads * 4) {
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int s = 0; s < a.n_splits; s++) {
+    const int nc = a.rank >> 2, ng = max(1, kMergeThreads / nc), gi = tid / nc, c = (tid - gi * nc) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (gi < ng) {
+#pragma unroll 8
+        for (int s = gi; s < a.n_splits; s += ng) {
             const float w = wsp[s];
-            if (w == 0.f) continue;  // an empty split has written no rows
-            const float4 x = load4(a.part_o + (part + s) * a.rank + c);
-            v.x = fmaf(w, x.x, v.x);
-            v.y = fmaf(w, x.y, v.y);
-            v.z = fmaf(w, x.z, v.z);
-            v.w = fmaf(w, x.w, v.w);
+            if (w != 0.f) {  // an empty split has written no rows
+                const float4 x = load4(a.part_o + (part + s) * a.rank + c);
+                v.x = fmaf(w, x.x, v.x);
+                v.y = fmaf(w, x.y, v.y);
+                v.z = fmaf(w, x.z, v.z);
+                v.w = fmaf(w, x.w, v.w);
+            }
         }
-        store4(ol + c, v);
+        store4(acc_s + tid * 4, v);
     }
     __syncthreads();
+    if (gi == 0) {
+        for (int k = 1; k < ng; k++) {
+            const float4 x = load4(acc_s + (k * nc + tid) * 4);
+            v.x += x.x;
+            v.y += x.y;
+            v.z += x.z;
+            v.w += x.w;
+        }
+        if (!wuv)
+            store4(static_cast<bf16 *>(a.out) + ((size_t)row * a.heads + h) * a.rank + c, v);
+        else
+            store4(ol + c, v);
+    }
+    if (!wuv) return;
+    __syncthreads();
     const float gate = sigmoid_f32(a.gate[(size_t)row * a.ld_gate + h]);
-    const int v0 = blockIdx.z * p.rows_per, v1 = min(a.vdim, v0 + p.rows_per);
-    for (int v = v0 + warp; v < v1; v += kMergeThreads / 32) {
-        const bf16 *w = static_cast<const bf16 *>(a.w_uv) + ((size_t)h * a.vdim + v) * a.rank;
+    for (int r = v0 + warp; r < v1; r += kMergeThreads / 32) {
+        const bf16 *w = wuv + ((size_t)h * a.vdim + r) * a.rank;
         float acc = 0.f;
-        for (int c = lane * 4; c < a.rank; c += 128) {
-            const float4 x = load4(w + c), y = load4(ol + c);
+#pragma unroll 4
+        for (int k = lane * 4; k < a.rank; k += 128) {
+            const float4 x = load4(w + k), y = load4(ol + k);
             acc = fmaf(x.x, y.x, acc);
             acc = fmaf(x.y, y.y, acc);
             acc = fmaf(x.z, y.z, acc);
@@ -259,7 +316,7 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const Merge
         }
 #pragma unroll
         for (int d = 16; d > 0; d >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, d);
-        if (lane == 0) static_cast<bf16 *>(a.out)[(size_t)row * a.heads * a.vdim + (size_t)h * a.vdim + v] = __float2bfloat16_rn(acc * gate);
+        if (lane == 0) static_cast<bf16 *>(a.out)[(size_t)row * a.heads * a.vdim + (size_t)h * a.vdim + r] = __float2bfloat16_rn(acc * gate);
     }
 }
 
@@ -279,23 +336,30 @@ __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_ke
     bf16 *qs = reinterpret_cast<bf16 *>(sm);
     bf16 *ks = qs + BR * kp;                 // [2][64][kp]
     bf16 *vs = ks + 2 * kFlKeys * kp;        // [2][64][vpitch]
-    const int h = blockIdx.y, r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * BR;  // long rows first
+    const int h = blockIdx.x, r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * BR;  // long rows first
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const bf16 *q = static_cast<const bf16 *>(a.q) + (size_t)h * dp;
     const bf16 *kv = static_cast<const bf16 *>(a.kv);
     const int ldq = a.heads * dp, rows = min(BR, a.n - r0), len = a.pos0 + r0 + rows;  // keys any row of the tile sees
     const int kc = dp >> 3, vc = vp >> 3;
+    // this thread's first (row, 16-byte piece) of a tile and the step to its next, for keys and values
+    const int kr0 = tid / kc, kch0 = tid - kr0 * kc, krs = kFlThreads / kc, kcs = kFlThreads - krs * kc;
+    const int vr0 = tid / vc, vch0 = tid - vr0 * vc, vrs = kFlThreads / vc, vcs = kFlThreads - vrs * vc;
+    auto load_rows = [&](const bf16 *src, uint32_t dst, int pitch, int j, int r, int ch, int rs, int chs, int nch) {
+        while (r < kFlKeys) {
+            const bool ok = j + r < len;
+            cp16(dst + (uint32_t)(r * pitch + ch * 8) * 2, src + (size_t)(ok ? j + r : 0) * a.ldkv + ch * 8, ok);
+            ch += chs;
+            r += rs;
+            if (ch >= nch) {
+                ch -= nch;
+                r++;
+            }
+        }
+    };
     auto load_kv = [&](int j, int buf) {
-        for (int i = tid; i < kFlKeys * kc; i += kFlThreads) {
-            const int r = i / kc, ch = i - r * kc;
-            const bool ok = j + r < len;
-            cp16(smem_addr(ks + ((size_t)buf * kFlKeys + r) * kp + ch * 8), kv + (size_t)(ok ? j + r : 0) * a.ldkv + h * dp + ch * 8, ok);
-        }
-        for (int i = tid; i < kFlKeys * vc; i += kFlThreads) {
-            const int r = i / vc, ch = i - r * vc;
-            const bool ok = j + r < len;
-            cp16(smem_addr(vs + ((size_t)buf * kFlKeys + r) * vpitch + ch * 8), kv + (size_t)(ok ? j + r : 0) * a.ldkv + a.heads * dp + h * vp + ch * 8, ok);
-        }
+        load_rows(kv + h * dp, smem_addr(ks + (size_t)buf * kFlKeys * kp), kp, j, kr0, kch0, krs, kcs, kc);
+        load_rows(kv + a.heads * dp + h * vp, smem_addr(vs + (size_t)buf * kFlKeys * vpitch), vpitch, j, vr0, vch0, vrs, vcs, vc);
         cp_commit();
     };
     for (int i = tid; i < BR * kc; i += kFlThreads) {
@@ -369,14 +433,14 @@ __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_ke
                 mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 1));
                 mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 2));
                 const float base = mv == -INFINITY ? 0.f : mv * p.scale_log2;
-                const float f = exp2f(mx[m][e2] * p.scale_log2 - base);
+                const float f = ex2(mx[m][e2] * p.scale_log2 - base);
                 mx[m][e2] = mv;
                 float sum = 0.f;
 #pragma unroll
                 for (int i = 0; i < kFlKeys / 8; i++)
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
-                        const float v = exp2f(fmaf(s[m][i][e2 * 2 + e], p.scale_log2, -base));
+                        const float v = ex2(fmaf(s[m][i][e2 * 2 + e], p.scale_log2, -base));
                         s[m][i][e2 * 2 + e] = v;
                         sum += v;
                     }
@@ -445,33 +509,45 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t *plane
 }
 
 // ───────────────────────────── launches ───────────────────────────────────────────────────
-static int head_groups(int heads) { return heads <= 16 ? 1 : (heads + 31) / 32; }
+// Heads of a CTA: 32 (two tensor-core row tiles) when there are that many and the shared memory holds them.
+static int head_tile(int heads, int rank) { return heads > 16 && rank <= 512 ? 32 : 16; }
+static int key_tile(int rank) { return rank <= 512 ? 64 : 32; }
 
-int latent_pick_splits(const juno_ctx *c, int n, int heads, int len_bound) {
-    const int want = std::max(1, 2 * c->sm_count / std::max(1, n * head_groups(heads)));
-    const int most = std::max(1, (len_bound + 2 * kSpKeys - 1) / (2 * kSpKeys));  // at least 64 positions each
-    return std::max(1, std::min(std::min(want, most), kMaxSplits));
+int latent_pick_splits(const juno_ctx *c, int n, int heads, int rank, int len_bound) {
+    const int ht = head_tile(heads, rank), kt = key_tile(rank), ctas = n * ((heads + ht - 1) / ht), tiles = (len_bound + kt - 1) / kt;
+    int best = 1;
+    double best_cost = 1e30;
+    for (int s = 1; s <= std::min(tiles, kMaxSplits); s++) {
+        // rounds of CTAs over the SMs, each as long as its tiles and a start-up; more splits cost the merge a little
+        const double waves = ((long long)ctas * s + c->sm_count - 1) / c->sm_count, cost = waves * ((tiles + s - 1) / s + 1.5) + 0.02 * s;
+        if (s > 1 && (long long)ctas * s > 2ll * c->sm_count + ctas) break;
+        if (cost < best_cost) {
+            best_cost = cost;
+            best = s;
+        }
+    }
+    return best;
 }
 size_t latent_part_floats(const juno_ctx *c, int n, int heads, int rank) {
-    const int groups = head_groups(heads);
-    return (size_t)std::min<long long>((long long)n * groups * kMaxSplits, 2ll * c->sm_count + (long long)n * groups) * (heads <= 16 ? 16 : 32) * (rank + 2);
+    const int ht = head_tile(heads, rank);
+    const long long groups = (long long)n * ((heads + ht - 1) / ht);
+    return (size_t)std::min(groups * kMaxSplits, 2ll * c->sm_count + groups) * ht * (rank + 2);
 }
 
-template <int MT, int NP>
+template <int MT, int KT, int NP>
 static int split_launch(juno_ctx *c, const SplitParams &p, int n, cudaStream_t st) {
     constexpr int HM = 16 * MT;
-    const size_t smem = (size_t)(HM + 2 * kSpKeys) * (p.rank + 8) * 2 + (size_t)HM * (kSpKeys + 8) * 2 + (size_t)4 * HM * (kSpKeys + 2) * 4 + (size_t)3 * HM * 4;
-    auto kernel = latent_split_kernel<MT, NP>;
+    const size_t smem = split_smem<MT, KT>(p.rank);
     static std::mutex mu;
     static size_t have[16] = {0};
     {
         std::lock_guard<std::mutex> lk(mu);
         if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(latent_split_kernel<MT, KT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             have[c->device & 15] = smem;
         }
     }
-    JUNO_CUDA_TRY(launch_pdl(kernel, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
+    JUNO_CUDA_TRY(launch_pdl(latent_split_kernel<MT, KT, NP>, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
     c->kernel_launches++;
     return JUNO_OK;
 }
@@ -494,20 +570,21 @@ int launch_latent_attn_split(juno_ctx *c, const LatentSplitArgs &a, cudaStream_t
     p.part_o = a.part_o;
     p.part_ml = a.part_ml;
     ProfScope prof(c, st, PROF_ATTN, 0);
-    const int n = a.rows.n, pw = ((a.rank >> 4) + kSpWarps - 1) / kSpWarps;
-    if (a.heads <= 16) return pw <= 1 ? split_launch<1, 1>(c, p, n, st) : pw <= 4 ? split_launch<1, 4>(c, p, n, st) : split_launch<1, 8>(c, p, n, st);
-    return pw <= 1 ? split_launch<2, 1>(c, p, n, st) : pw <= 4 ? split_launch<2, 4>(c, p, n, st) : split_launch<2, 8>(c, p, n, st);
+    const int n = a.rows.n;
+    if (a.rank > 512) return split_launch<1, 32, 4>(c, p, n, st);
+    if (a.heads <= 16) return a.rank <= 256 ? split_launch<1, 64, 1>(c, p, n, st) : split_launch<1, 64, 2>(c, p, n, st);
+    return a.rank <= 256 ? split_launch<2, 64, 1>(c, p, n, st) : split_launch<2, 64, 2>(c, p, n, st);
 }
 
 int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st) {
     JUNO_REQUIRE(a.n > 0 && a.heads > 0 && a.rank % 16 == 0 && a.rank <= kLatentSplitMaxRank && a.n_splits >= 1 && a.n_splits <= kMaxSplits, "latent merge: bad arguments");
     MergeParams p;
     p.a = a;
-    int parts = std::max(1, std::min((a.vdim + 15) / 16, (c->sm_count + a.n * a.heads - 1) / (a.n * a.heads)));
+    int parts = a.w_uv ? std::max(1, std::min((a.vdim + 15) / 16, (c->sm_count + a.n * a.heads - 1) / (a.n * a.heads))) : 1;
     p.rows_per = (a.vdim + parts - 1) / parts;
     parts = (a.vdim + p.rows_per - 1) / p.rows_per;
     ProfScope prof(c, st, PROF_ATTN, 0);
-    JUNO_CUDA_TRY(launch_pdl(latent_merge_kernel, dim3((unsigned)a.heads, (unsigned)a.n, (unsigned)parts), dim3(kMergeThreads), (size_t)a.rank * 4, st, p));
+    JUNO_CUDA_TRY(launch_pdl(latent_merge_kernel, dim3((unsigned)a.heads, (unsigned)a.n, (unsigned)parts), dim3(kMergeThreads), 0, st, p));
     c->kernel_launches++;
     return JUNO_OK;
 }
@@ -525,7 +602,7 @@ static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
             have[c->device & 15] = smem;
         }
     }
-    flash_prefill_kernel<D, MT><<<dim3((unsigned)((p.a.n + BR - 1) / BR), (unsigned)p.a.heads), kFlThreads, smem, st>>>(p);
+    flash_prefill_kernel<D, MT><<<dim3((unsigned)p.a.heads, (unsigned)((p.a.n + BR - 1) / BR)), kFlThreads, smem, st>>>(p);
     JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;

@@ -147,6 +147,48 @@ __global__ void __launch_bounds__(128) conv_kernel(const ConvParams p) {
     }
 }
 
+// A portion of a prompt: the window of the last TAPS inputs stays in registers while a thread walks down its rows.
+constexpr int kConvSeqRows = 16;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) conv_seq_kernel(const ConvParams p) {
+    const int col = (blockIdx.x * 128 + threadIdx.x) * 4;
+    if (col >= p.ldx) return;
+    const T *w = static_cast<const T *>(p.w);
+    float4 wv[TAPS], win[TAPS];  // win[k]: the input k positions back
+#pragma unroll
+    for (int k = 0; k < TAPS; k++) wv[k] = load4(w + (size_t)(TAPS - 1 - k) * p.ldx + col);
+    const int r0 = blockIdx.y * kConvSeqRows, r1 = min(p.n, r0 + kConvSeqRows);
+    const int pos0 = p.positions[r0];
+    auto input = [&](int r) {
+        const float4 v = load4(p.x + (size_t)r * p.ldx + col);
+        const float s = p.row_scale[r];
+        return make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
+    };
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; k++) {
+        const int back = k + 1;  // before row r0
+        win[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (back <= pos0)
+            win[k] = back <= r0 ? input(r0 - back)
+                                : load4(p.state + (size_t)p.slots[r0] * p.slot_stride + (size_t)((pos0 - back) & p.ring_mask) * p.ldx + col);
+    }
+#pragma unroll 4
+    for (int r = r0; r < r1; r++) {
+#pragma unroll
+        for (int k = TAPS - 1; k > 0; k--) win[k] = win[k - 1];
+        const float4 h = win[0] = input(r);
+        float4 acc = h;
+#pragma unroll
+        for (int k = 0; k < TAPS; k++) {
+            acc.x = fmaf(wv[k].x, win[k].x, acc.x);
+            acc.y = fmaf(wv[k].y, win[k].y, acc.y);
+            acc.z = fmaf(wv[k].z, win[k].z, acc.z);
+            acc.w = fmaf(wv[k].w, win[k].w, acc.w);
+        }
+        store4(static_cast<T *>(p.out) + (size_t)r * p.ldo + col, acc);
+    }
+}
+
 // After a portion: its last inputs into the state (a launch of its own, because the portion's first rows still read the
 // entries that its last rows replace).
 __global__ void __launch_bounds__(128) conv_state_kernel(const ConvParams p) {
@@ -254,8 +296,15 @@ int launch_conv(juno_ctx *c, int dt, const ConvArgs &a, const RowSet &rows, cuda
     const unsigned gx = (unsigned)((a.ldx + 511) / 512);
     const dim3 grid(gx, (unsigned)((rows.n + kConvRows - 1) / kConvRows));
     ProfScope prof(c, st, PROF_ROWOPS, (double)rows.n * a.width * (4 + dt_bytes(dt)));
+    const dim3 sgrid(gx, (unsigned)((rows.n + kConvSeqRows - 1) / kConvSeqRows));
     if (dt == DT_F32)
         conv_kernel<float><<<grid, 128, 0, st>>>(p);
+    else if (rows.one_seq && a.taps == 2)
+        conv_seq_kernel<bf16, 2><<<sgrid, 128, 0, st>>>(p);
+    else if (rows.one_seq && a.taps == 3)
+        conv_seq_kernel<bf16, 3><<<sgrid, 128, 0, st>>>(p);
+    else if (rows.one_seq && a.taps == 4)
+        conv_seq_kernel<bf16, 4><<<sgrid, 128, 0, st>>>(p);
     else
         conv_kernel<bf16><<<grid, 128, 0, st>>>(p);
     JUNO_CUDA_TRY(cudaGetLastError());

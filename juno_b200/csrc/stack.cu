@@ -99,6 +99,7 @@ int stack_upload_f32(juno_ctx *c, StackNet *net, const std::vector<float> &v, fl
 // A portion of a prompt with at most this many positions attends with absorbed queries, like a decode step: expanding keys and
 // values from the whole context would cost more than it saves.
 constexpr int kAbsorbRows = 48;
+constexpr int kMergeRows = 8;  // rows up to which the value projection is done by the merge of the context splits
 static bool flash_fits(const LatentMixerSpec &m) { return m.dp() <= kFlashMaxDim && m.vp() <= kFlashMaxDim; }
 
 // ───────────────────────────── buffers ────────────────────────────────────────────────────
@@ -189,11 +190,17 @@ void stack_step_done(const juno_ctx *c, StackNet *net, int n) {
 
 const float *stack_residual(const StackNet *net) { return net->last_x ? net->x2 : net->x; }
 
+// One split count for all layers of a step (it is part of the captured step's key): the largest any layer's shape asks for
+// that every layer's buffers and kernels take.
 int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bound) {
     if (net->dt != DT_BF16) return 1;
-    int heads = 1;
-    for (const StackLayerSpec &L : net->spec.layers) heads = std::max(heads, L.mix.heads);
-    return latent_pick_splits(c, n, heads, len_bound);
+    int best = 1, most = 1 << 30;
+    for (const StackLayerSpec &L : net->spec.layers) {
+        if (L.mix.rp() > kLatentSplitMaxRank) continue;
+        best = std::max(best, latent_pick_splits(c, n, L.mix.heads, L.mix.rp(), len_bound));
+        most = std::min<long long>(most, (long long)(net->part_floats / ((size_t)n * L.mix.heads * (L.mix.rp() + 2))));
+    }
+    return std::max(1, std::min(best, most));
 }
 
 // ───────────────────────────── attention of one layer ─────────────────────────────────────
@@ -243,11 +250,14 @@ static int attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, con
         JUNO_REQUIRE(ml + (size_t)n * H * n_splits * 2 <= net->part_floats, "%d context splits of %d rows exceed the buffer", n_splits, n);
         LatentSplitArgs sp{pool, layer, rows, H, rp, n_splits, m.scale, net->qlat, net->part_o, net->part_o + ml};
         JUNO_TRY(launch_latent_attn_split(c, sp, st));
-        LatentMergeArgs mg{n, H, rp, vp, n_splits, net->part_o, net->part_o + ml, w_uv, gate, net->ldu, net->att};
-        return launch_latent_merge(c, mg, st);
+        const bool fold = n <= kMergeRows;  // the value projection inside the merge reads W_uv once per row
+        LatentMergeArgs mg{n, H, rp, vp, n_splits, net->part_o, net->part_o + ml, fold ? w_uv : nullptr, gate, net->ldu, fold ? net->att : net->olat};
+        JUNO_TRY(launch_latent_merge(c, mg, st));
+        if (fold) return JUNO_OK;
+    } else {
+        LatentAttnArgs at{pool, layer, rows, H, rp, m.scale, net->qlat, net->olat};
+        JUNO_TRY(launch_latent_attn_simt(c, dt, at, st));
     }
-    LatentAttnArgs at{pool, layer, rows, H, rp, m.scale, net->qlat, net->olat};
-    JUNO_TRY(launch_latent_attn_simt(c, dt, at, st));
     g.a = net->olat;
     g.lda = H * rp;
     g.w = w_uv;
