@@ -205,6 +205,20 @@ def workload_config(args, arch):
             "l2": "weights read per step (GBs) exceed the 126 MB L2; no explicit flush"}
 
 
+def run_design(args):
+    import torch
+    from juno_b200 import stackbench
+    torch.cuda.set_device(0)
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    peaks = json.load(open(p)) if os.path.exists(p) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = stackbench.run(args.sizes.split(","), [int(b) for b in args.batches.split(",")], args.ctx, args.steps, args.warmup,
+                         {k: float(peaks[k]) for k in ("hbm_gbs", "bf16_tflops")}, not args.no_llama)
+    print(json.dumps({"design": args.design, "context": args.ctx, "steps": args.steps, "warmup": args.warmup, "data": "synthetic",
+                      "dtype": "bf16", "clocks": sampler.result(), "sizes": res}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -218,7 +232,15 @@ def main():
     ap.add_argument("--no-prefill", action="store_true", help="start decoding at an empty context (quick runs)")
     ap.add_argument("--chunked-prefill", action="store_true",
                     help="fill the prompt through juno_prefill (batched kernels, up to 64 positions per pass) instead of token by token")
+    ap.add_argument("--design", choices=["vosotar"], help="instead of the default workload: prefill and decode of a registered design "
+                    "beside the LLaMA family at equal size (one GPU, one JSON line)")
+    ap.add_argument("--sizes", default="small,medium,large", help="with --design")
+    ap.add_argument("--batches", default="1,8,64", help="with --design: decode batches")
+    ap.add_argument("--no-llama", action="store_true", help="with --design: the design alone")
     args = ap.parse_args()
+    if args.design:
+        run_design(args)
+        return
     arch, seed = MODELS[args.model]
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

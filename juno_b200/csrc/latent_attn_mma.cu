@@ -12,10 +12,11 @@ using bf16 = __nv_bfloat16;
 constexpr float kLog2e = 1.4426950408889634f;
 
 // ───────────────────────────── decode: splits of the context ──────────────────────────────
-// A CTA (sixteen warps, one per SM) takes a group of 16 * MT heads of one row and a range of positions, KT at a time, the next
-// tile in flight.  Scores: warp (16 positions, part of the rank) multiplies its part of q_lat with the tile, the parts are added
-// in shared memory; online softmax by rows; then each warp owns a range of latent columns of O += P C, reading the same tile
-// transposed.
+// A CTA (sixteen warps, one per SM) takes a group of 16 * MT heads of one row and a range of positions, 32 at a time.  Scores:
+// warp (16 positions, an eighth of the rank) multiplies its part of q_lat - A fragments it keeps in registers - with the tile,
+// the eight parts are added in shared memory; online softmax by rows; O += P C: each warp owns a range of latent columns and
+// reads the tile transposed.  The scores of tile i + 1 and the averages of tile i are one phase between barriers (their MMAs
+// fill each other's latencies), while tile i + 2 is on its way.
 constexpr int kSpThreads = 512, kSpWarps = 16;
 
 struct SplitParams {
@@ -33,29 +34,36 @@ __device__ __forceinline__ float ex2(float v) {
     return r;
 }
 
-template <int MT, int KT>
-constexpr size_t split_smem(int rank) {
-    return (size_t)(16 * MT + 2 * KT) * (rank + 8) * 2 + (size_t)16 * MT * (KT + 8) * 2 + (size_t)(kSpWarps * 16 / KT) * 16 * MT * (KT + 2) * 4 +
-           (size_t)3 * 16 * MT * 4;
+__device__ __forceinline__ float warp_max(float v) {
+    float r;
+    asm("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
+    return r;
 }
 
-template <int MT, int KT, int NP>  // NP: 16-column pairs of n-tiles a warp owns at most
+constexpr int kSpKeys = 32, kSpParts = 8, kSpPitch = kSpKeys + 8;  // score rows 8 banks apart: the float2 stores of a warp meet no bank twice
+
+template <int MT>
+constexpr size_t split_smem(int rank) {
+    return (size_t)3 * kSpKeys * (rank + 8) * 2 + (size_t)16 * MT * (kSpKeys + 8) * 2 + (size_t)kSpParts * 16 * MT * kSpPitch * 4 + (size_t)16 * MT * 4;
+}
+
+// NQ: 16-column steps of the rank a warp scores at most; NP: 16-column pairs of n-tiles a warp averages at most
+template <int MT, int NQ, int NP>
 __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const SplitParams p) {
     extern __shared__ __align__(16) uint8_t sm[];
-    constexpr int HM = 16 * MT, KG = KT / 16, RQ = kSpWarps / KG, SP = KT + 2;
+    constexpr int HM = 16 * MT, SP = kSpPitch;
     const int R = p.rank, pitch = R + 8;
-    bf16 *qs = reinterpret_cast<bf16 *>(sm);          // [HM][pitch]
-    bf16 *cs = qs + HM * pitch;                       // [2][KT][pitch]
-    bf16 *ps = cs + 2 * KT * pitch;                   // [HM][KT + 8]
-    float *ss = reinterpret_cast<float *>(ps + HM * (KT + 8));  // [RQ][HM][SP]
-    float *fac = ss + RQ * HM * SP, *mrow = fac + HM, *lrow = mrow + HM;
+    bf16 *cs = reinterpret_cast<bf16 *>(sm);          // [3][kSpKeys][pitch]
+    bf16 *ps = cs + 3 * kSpKeys * pitch;              // [HM][kSpKeys + 8]
+    float *ss = reinterpret_cast<float *>(ps + HM * (kSpKeys + 8));  // [kSpParts][HM][SP]
+    float *fac = ss + kSpParts * HM * SP;
     const int split = blockIdx.x, h0 = blockIdx.y * HM, row = blockIdx.z, nh = min(HM, p.heads - h0);
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     pdl_wait();
     pdl_launch_dependents();
     const int len = p.positions[row] + 1;
-    const int tiles = (len + KT - 1) / KT, per = (tiles + p.n_splits - 1) / p.n_splits;
-    const int j0 = split * per * KT, j1 = min(len, j0 + per * KT);
+    const int tiles = (len + kSpKeys - 1) / kSpKeys, per = (tiles + p.n_splits - 1) / p.n_splits;
+    const int j0 = split * per * kSpKeys, j1 = min(len, j0 + per * kSpKeys);
     const size_t part = ((size_t)row * p.heads + h0) * p.n_splits + split;  // + head * n_splits
     if (j0 >= j1) {
         if (tid < nh) {
@@ -66,36 +74,39 @@ __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const Split
     }
     const int32_t *table = p.table + (size_t)p.slots[row] * p.max_pages;
     const int chunks = R >> 3;
-    // KT / 16 consecutive rows per warp: they lie in one page
-    constexpr int WR = KT / kSpWarps;
+    const int r0 = warp * 2;  // two consecutive rows per warp: they lie in one page, whose number is read a tile ahead
+    auto page_of = [&](int j) { return j + r0 < j1 ? table[(j + r0) >> 4] : 0; };
+    int page = page_of(j0);
     auto load_tile = [&](int j, int buf) {
-        const int r0 = warp * WR;
-        const bool any = j + r0 < j1;
-        const bf16 *src = any ? latent_row(p.plane, table, R, j + r0) : p.plane;
-        const uint32_t dst = smem_addr(cs + ((size_t)buf * KT + r0) * pitch);
+        const bf16 *src = p.plane + ((size_t)page * kPageTokens + ((j + r0) & (kPageTokens - 1))) * R;
+        page = page_of(j + kSpKeys);
+        const uint32_t dst = smem_addr(cs + ((size_t)buf * kSpKeys + r0) * pitch);
 #pragma unroll
-        for (int i = 0; i < WR; i++) {
+        for (int i = 0; i < 2; i++) {
             const bool ok = j + r0 + i < j1;
             for (int ch = lane; ch < chunks; ch += 32) cp16(dst + (uint32_t)(i * pitch + ch * 8) * 2, ok ? src + (size_t)i * R + ch * 8 : p.plane, ok);
         }
         cp_commit();
     };
-    {
-        const bf16 *q = p.q + ((size_t)row * p.heads + h0) * R;
-        for (int r = warp; r < HM; r += kSpWarps) {
-            const bool ok = r < nh;
-            for (int ch = lane; ch < chunks; ch += 32) cp16(smem_addr(qs + r * pitch + ch * 8), ok ? q + (size_t)r * R + ch * 8 : q, ok);
-        }
-    }
     load_tile(j0, 0);
-    if (tid < HM) {
-        mrow[tid] = -INFINITY;
-        lrow[tid] = 0.f;
-    }
-    const int kg = warp % KG, rq = warp / KG;                     // 16 positions, part of the rank
-    const int ksteps = R >> 4, ks0 = ksteps * rq / RQ, ks1 = ksteps * (rq + 1) / RQ;
+    if (j0 + kSpKeys < j1)
+        load_tile(j0 + kSpKeys, 1);
+    else
+        cp_commit();
+    const int kg = warp & 1, rq = warp >> 1;                      // 16 positions, part of the rank
+    const int ksteps = R >> 4, ks0 = ksteps * rq / kSpParts, nq = ksteps * (rq + 1) / kSpParts - ks0;
     const int pairs = R >> 4, pw = (pairs + kSpWarps - 1) / kSpWarps, c0 = warp * pw * 16;  // columns of O
     const int np = max(0, min(pw, pairs - warp * pw));
+    uint32_t qa[NQ][MT][4];
+#pragma unroll
+    for (int k = 0; k < NQ; k++)
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int r = m * 16 + g + (e & 1) * 8, col = (ks0 + k) * 16 + 2 * t + (e >> 1) * 8;
+                qa[k][m][e] = k < nq && r < nh ? *reinterpret_cast<const uint32_t *>(p.q + ((size_t)row * p.heads + h0 + r) * R + col) : 0u;
+            }
     float o[MT][NP][2][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
@@ -107,80 +118,64 @@ __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const Split
                 for (int e = 0; e < 4; e++) o[m][i][k][e] = 0.f;
     const int lr = lane & 15, lc = (lane >> 4) * 8;   // ldmatrix x4: row, column offset (A operand; transposed B operand)
     const int br = (lane & 7) + (lane >> 4) * 8, bc = ((lane >> 3) & 1) * 8;  // B operand from rows of keys: two n-tiles at once
-    const int g = lane >> 2, t = lane & 3;
-    const uint32_t q_a = smem_addr(qs + lr * pitch + lc), p_a = smem_addr(ps + lr * (KT + 8) + lc);
-    int buf = 0;
-    for (int j = j0; j < j1; j += KT, buf ^= 1) {
-        cp_wait<0>();
-        __syncthreads();
-        if (j + KT < j1) load_tile(j + KT, buf ^ 1);
-        const bf16 *ct = cs + (size_t)buf * KT * pitch;
-        {
-            float s[MT][2][4];
+    const uint32_t p_a = smem_addr(ps + lr * (kSpKeys + 8) + lc);
+    const uint32_t cs_a = smem_addr(cs), k_off = (uint32_t)((kg * 16 + br) * pitch + ks0 * 16 + bc) * 2, v_off = (uint32_t)(lr * pitch + c0 + lc) * 2;
+    const uint32_t tile_bytes = (uint32_t)kSpKeys * pitch * 2;
+    auto scores = [&](int buf) {
+        float s[MT][2][4];
 #pragma unroll
-            for (int m = 0; m < MT; m++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-                for (int k = 0; k < 2; k++)
+            for (int k = 0; k < 2; k++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) s[m][k][e] = 0.f;
-            const uint32_t k_a = smem_addr(ct + (kg * 16 + br) * pitch + bc);
-#pragma unroll 4
-            for (int ks = ks0; ks < ks1; ks++) {
+                for (int e = 0; e < 4; e++) s[m][k][e] = 0.f;
+#pragma unroll
+        for (int k = 0; k < NQ; k++)
+            if (k < nq) {
                 uint32_t b[4];
-                ldsm4(b, k_a + ks * 32);
+                ldsm4(b, cs_a + buf * tile_bytes + k_off + k * 32);
 #pragma unroll
                 for (int m = 0; m < MT; m++) {
-                    uint32_t a[4];
-                    ldsm4(a, q_a + (uint32_t)(m * 16 * pitch + ks * 16) * 2);
-                    mma16816(s[m][0], a, b[0], b[1]);
-                    mma16816(s[m][1], a, b[2], b[3]);
+                    mma16816(s[m][0], qa[k][m], b[0], b[1]);
+                    mma16816(s[m][1], qa[k][m], b[2], b[3]);
                 }
             }
 #pragma unroll
-            for (int m = 0; m < MT; m++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-                for (int k = 0; k < 2; k++) {
-                    float *d = ss + (rq * HM + m * 16 + g) * SP + kg * 16 + k * 8 + 2 * t;
-                    *reinterpret_cast<float2 *>(d) = make_float2(s[m][k][0], s[m][k][1]);
-                    *reinterpret_cast<float2 *>(d + 8 * SP) = make_float2(s[m][k][2], s[m][k][3]);
-                }
+            for (int k = 0; k < 2; k++) {
+                float *d = ss + (rq * HM + m * 16 + g) * SP + kg * 16 + k * 8 + 2 * t;
+                *reinterpret_cast<float2 *>(d) = make_float2(s[m][k][0], s[m][k][1]);
+                *reinterpret_cast<float2 *>(d + 8 * SP) = make_float2(s[m][k][2], s[m][k][3]);
+            }
+    };
+    // a warp's MT rows are always the same ones: running maximum (the same in all lanes) and each lane's share of the sum
+    float run_m[MT], run_l[MT];
+#pragma unroll
+    for (int i = 0; i < MT; i++) {
+        run_m[i] = -INFINITY;
+        run_l[i] = 0.f;
+    }
+    auto softmax = [&](int j) {
+        float v[MT];
+#pragma unroll
+        for (int i = 0; i < MT; i++) v[i] = 0.f;
+#pragma unroll
+        for (int k = 0; k < kSpParts; k++)
+#pragma unroll
+            for (int i = 0; i < MT; i++) v[i] += ss[(k * HM + warp * MT + i) * SP + lane];
+#pragma unroll
+        for (int i = 0; i < MT; i++) {
+            const int r = warp * MT + i;
+            v[i] = j + lane < j1 ? v[i] * p.scale_log2 : -INFINITY;
+            const float m = fmaxf(run_m[i], warp_max(v[i])), f = ex2(run_m[i] - m), e = ex2(v[i] - m);
+            ps[r * (kSpKeys + 8) + lane] = __float2bfloat16_rn(e);
+            if (lane == 0) fac[r] = f;
+            run_l[i] = run_l[i] * f + e;
+            run_m[i] = m;
         }
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < HM / kSpWarps; i++) {
-            const int r = warp * (HM / kSpWarps) + i;
-            float v[KT / 32];
-            float m = -INFINITY;
-#pragma unroll
-            for (int x = 0; x < KT / 32; x++) {
-                v[x] = 0.f;
-#pragma unroll
-                for (int k = 0; k < RQ; k++) v[x] += ss[(k * HM + r) * SP + x * 32 + lane];
-                v[x] = j + x * 32 + lane < j1 ? v[x] * p.scale_log2 : -INFINITY;
-                m = fmaxf(m, v[x]);
-            }
-#pragma unroll
-            for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
-            const float mo = mrow[r];
-            m = fmaxf(m, mo);
-            float sum = 0.f;
-#pragma unroll
-            for (int x = 0; x < KT / 32; x++) {
-                const float e = ex2(v[x] - m);
-                sum += e;
-                ps[r * (KT + 8) + x * 32 + lane] = __float2bfloat16_rn(e);
-            }
-#pragma unroll
-            for (int d = 16; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-            __syncwarp();
-            if (lane == 0) {
-                const float f = ex2(mo - m);
-                fac[r] = f;
-                lrow[r] = lrow[r] * f + sum;
-                mrow[r] = m;
-            }
-        }
-        __syncthreads();
+    };
+    auto averages = [&](int buf) {
 #pragma unroll
         for (int m = 0; m < MT; m++) {
             const float f0 = fac[m * 16 + g], f1 = fac[m * 16 + g + 8];
@@ -194,27 +189,42 @@ __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const Split
                     o[m][i][k][3] *= f1;
                 }
         }
-        const uint32_t v_a = smem_addr(ct + lr * pitch + c0 + lc);
 #pragma unroll
-        for (int kk = 0; kk < KT / 16; kk++) {
+        for (int kk = 0; kk < kSpKeys / 16; kk++) {
             uint32_t a[MT][4];
 #pragma unroll
-            for (int m = 0; m < MT; m++) ldsm4(a[m], p_a + (uint32_t)(m * 16 * (KT + 8) + kk * 16) * 2);
+            for (int m = 0; m < MT; m++) ldsm4(a[m], p_a + (uint32_t)(m * 16 * (kSpKeys + 8) + kk * 16) * 2);
 #pragma unroll
-            for (int i = 0; i < NP; i++) {
+            for (int i = 0; i < NP; i++)
                 if (i < np) {
                     uint32_t b[4];
-                    ldsm4_trans(b, v_a + (uint32_t)(kk * 16 * pitch + i * 16) * 2);
+                    ldsm4_trans(b, cs_a + buf * tile_bytes + v_off + (uint32_t)(kk * 16 * pitch + i * 16) * 2);
 #pragma unroll
                     for (int m = 0; m < MT; m++) {
                         mma16816(o[m][i][0], a[m], b[0], b[1]);
                         mma16816(o[m][i][1], a[m], b[2], b[3]);
                     }
                 }
-            }
         }
-    }
+    };
+    cp_wait<1>();
     __syncthreads();
+    scores(0);
+    __syncthreads();
+    softmax(j0);
+    int buf = 0;
+    for (int j = j0; j < j1; j += kSpKeys) {  // tile j has its weights in ps
+        const int b1 = buf == 2 ? 0 : buf + 1, b2 = b1 == 2 ? 0 : b1 + 1;
+        cp_wait<0>();
+        __syncthreads();
+        if (j + 2 * kSpKeys < j1) load_tile(j + 2 * kSpKeys, b2);
+        if (j + kSpKeys < j1) scores(b1);
+        averages(buf);
+        if (j + kSpKeys >= j1) break;
+        __syncthreads();
+        softmax(j + kSpKeys);
+        buf = b1;
+    }
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
@@ -226,9 +236,13 @@ __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const Split
                     if (ha < nh) *reinterpret_cast<float2 *>(p.part_o + (part + (size_t)ha * p.n_splits) * R + col) = make_float2(o[m][i][k][0], o[m][i][k][1]);
                     if (hb < nh) *reinterpret_cast<float2 *>(p.part_o + (part + (size_t)hb * p.n_splits) * R + col) = make_float2(o[m][i][k][2], o[m][i][k][3]);
                 }
-    if (tid < nh) {
-        p.part_ml[(part + (size_t)tid * p.n_splits) * 2] = mrow[tid];
-        p.part_ml[(part + (size_t)tid * p.n_splits) * 2 + 1] = lrow[tid];
+#pragma unroll
+    for (int i = 0; i < MT; i++) {
+        const int r = warp * MT + i;
+        float l = run_l[i];
+#pragma unroll
+        for (int d = 16; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+        if (lane == 0 && r < nh) *reinterpret_cast<float2 *>(p.part_ml + (part + (size_t)r * p.n_splits) * 2) = make_float2(run_m[i], l);
     }
 }
 
@@ -249,11 +263,6 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const Merge
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int v0 = blockIdx.z * p.rows_per, v1 = min(a.vdim, v0 + p.rows_per);
     const bf16 *wuv = static_cast<const bf16 *>(a.w_uv);
-    if (wuv)  // weights do not depend on the attention: on their way to L2 before it has finished
-        for (int i = tid; i < (v1 - v0) * a.rank / 64; i += kMergeThreads)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(wuv + ((size_t)h * a.vdim + v0) * a.rank + (size_t)i * 64));
-    pdl_wait();
-    pdl_launch_dependents();
     const size_t part = ((size_t)row * a.heads + h) * a.n_splits;
     if (warp == 0) {
         const bool h0 = lane < a.n_splits, h1 = lane + 32 < a.n_splits;
@@ -511,15 +520,14 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t *plane
 // ───────────────────────────── launches ───────────────────────────────────────────────────
 // Heads of a CTA: 32 (two tensor-core row tiles) when there are that many and the shared memory holds them.
 static int head_tile(int heads, int rank) { return heads > 16 && rank <= 512 ? 32 : 16; }
-static int key_tile(int rank) { return rank <= 512 ? 64 : 32; }
 
 int latent_pick_splits(const juno_ctx *c, int n, int heads, int rank, int len_bound) {
-    const int ht = head_tile(heads, rank), kt = key_tile(rank), ctas = n * ((heads + ht - 1) / ht), tiles = (len_bound + kt - 1) / kt;
+    const int ht = head_tile(heads, rank), ctas = n * ((heads + ht - 1) / ht), tiles = (len_bound + kSpKeys - 1) / kSpKeys;
     int best = 1;
     double best_cost = 1e30;
     for (int s = 1; s <= std::min(tiles, kMaxSplits); s++) {
         // rounds of CTAs over the SMs, each as long as its tiles and a start-up; more splits cost the merge a little
-        const double waves = ((long long)ctas * s + c->sm_count - 1) / c->sm_count, cost = waves * ((tiles + s - 1) / s + 1.5) + 0.02 * s;
+        const double waves = ((long long)ctas * s + c->sm_count - 1) / c->sm_count, cost = waves * ((tiles + s - 1) / s + 3) + 0.04 * s;
         if (s > 1 && (long long)ctas * s > 2ll * c->sm_count + ctas) break;
         if (cost < best_cost) {
             best_cost = cost;
@@ -534,20 +542,20 @@ size_t latent_part_floats(const juno_ctx *c, int n, int heads, int rank) {
     return (size_t)std::min(groups * kMaxSplits, 2ll * c->sm_count + groups) * ht * (rank + 2);
 }
 
-template <int MT, int KT, int NP>
+template <int MT, int NQ, int NP>
 static int split_launch(juno_ctx *c, const SplitParams &p, int n, cudaStream_t st) {
     constexpr int HM = 16 * MT;
-    const size_t smem = split_smem<MT, KT>(p.rank);
+    const size_t smem = split_smem<MT>(p.rank);
     static std::mutex mu;
     static size_t have[16] = {0};
     {
         std::lock_guard<std::mutex> lk(mu);
         if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(latent_split_kernel<MT, KT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(latent_split_kernel<MT, NQ, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             have[c->device & 15] = smem;
         }
     }
-    JUNO_CUDA_TRY(launch_pdl(latent_split_kernel<MT, KT, NP>, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
+    JUNO_CUDA_TRY(launch_pdl(latent_split_kernel<MT, NQ, NP>, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
     c->kernel_launches++;
     return JUNO_OK;
 }
@@ -571,9 +579,9 @@ int launch_latent_attn_split(juno_ctx *c, const LatentSplitArgs &a, cudaStream_t
     p.part_ml = a.part_ml;
     ProfScope prof(c, st, PROF_ATTN, 0);
     const int n = a.rows.n;
-    if (a.rank > 512) return split_launch<1, 32, 4>(c, p, n, st);
-    if (a.heads <= 16) return a.rank <= 256 ? split_launch<1, 64, 1>(c, p, n, st) : split_launch<1, 64, 2>(c, p, n, st);
-    return a.rank <= 256 ? split_launch<2, 64, 1>(c, p, n, st) : split_launch<2, 64, 2>(c, p, n, st);
+    if (a.rank > 512) return split_launch<1, 8, 4>(c, p, n, st);
+    if (a.heads <= 16) return a.rank <= 256 ? split_launch<1, 2, 1>(c, p, n, st) : split_launch<1, 4, 2>(c, p, n, st);
+    return a.rank <= 256 ? split_launch<2, 2, 1>(c, p, n, st) : split_launch<2, 4, 2>(c, p, n, st);
 }
 
 int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st) {
@@ -584,7 +592,10 @@ int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st) 
     p.rows_per = (a.vdim + parts - 1) / parts;
     parts = (a.vdim + p.rows_per - 1) / p.rows_per;
     ProfScope prof(c, st, PROF_ATTN, 0);
-    JUNO_CUDA_TRY(launch_pdl(latent_merge_kernel, dim3((unsigned)a.heads, (unsigned)a.n, (unsigned)parts), dim3(kMergeThreads), 0, st, p));
+    // an ordinary launch: its many small blocks, made resident early by a programmatic dependent launch, measured 70 us per
+    // layer slower at two and more sequences (they keep the large CTAs on both sides from their SMs)
+    latent_merge_kernel<<<dim3((unsigned)a.heads, (unsigned)a.n, (unsigned)parts), kMergeThreads, 0, st>>>(p);
+    JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;
 }
