@@ -74,8 +74,9 @@ def residual_gate(h, w, name):
 
 
 def layer(x, cfg, i, w):
-    spec = cfg["layers"][i]
-    src = spec.get("weights_of", i)
+    spec, src = cfg["layers"][i], i
+    while cfg["layers"][src].get("weights_of") is not None:  # this layer runs with another layer's tensors
+        src = cfg["layers"][src]["weights_of"]
     L, eps = f"l{src}.", cfg["norm"]["eps"]
     h = scalar_norm(x, w[L + "norm1"], eps)
     y = latent_attention(h + causal_conv(h, w[L + "canon1"]), spec["mixer"], w, L + "mix.", eps)
