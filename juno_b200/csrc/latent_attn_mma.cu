@@ -47,12 +47,13 @@ constexpr size_t split_smem(int rank) {
     return (size_t)3 * kSpKeys * (rank + 8) * 2 + (size_t)16 * MT * (kSpKeys + 8) * 2 + (size_t)kSpParts * 16 * MT * kSpPitch * 4 + (size_t)16 * MT * 4;
 }
 
-// NQ: 16-column steps of the rank a warp scores at most; NP: 16-column pairs of n-tiles a warp averages at most
-template <int MT, int NQ, int NP>
+// NQ: 16-column steps of the rank a warp scores at most; NP: 16-column pairs of n-tiles a warp averages at most; RANK: the rank,
+// when it is a common one (every offset and bound folds), else 0
+template <int MT, int NQ, int NP, int RANK>
 __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const SplitParams p) {
     extern __shared__ __align__(16) uint8_t sm[];
     constexpr int HM = 16 * MT, SP = kSpPitch;
-    const int R = p.rank, pitch = R + 8;
+    const int R = RANK ? RANK : p.rank, pitch = R + 8;
     bf16 *cs = reinterpret_cast<bf16 *>(sm);          // [3][kSpKeys][pitch]
     bf16 *ps = cs + 3 * kSpKeys * pitch;              // [HM][kSpKeys + 8]
     float *ss = reinterpret_cast<float *>(ps + HM * (kSpKeys + 8));  // [kSpParts][HM][SP]
@@ -179,6 +180,7 @@ __global__ void __launch_bounds__(kSpThreads, 1) latent_split_kernel(const Split
 #pragma unroll
         for (int m = 0; m < MT; m++) {
             const float f0 = fac[m * 16 + g], f1 = fac[m * 16 + g + 8];
+            if (!__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) continue;  // no maximum has moved
 #pragma unroll
             for (int i = 0; i < NP; i++)
 #pragma unroll
@@ -542,7 +544,7 @@ size_t latent_part_floats(const juno_ctx *c, int n, int heads, int rank) {
     return (size_t)std::min(groups * kMaxSplits, 2ll * c->sm_count + groups) * ht * (rank + 2);
 }
 
-template <int MT, int NQ, int NP>
+template <int MT, int NQ, int NP, int RANK = 0>
 static int split_launch(juno_ctx *c, const SplitParams &p, int n, cudaStream_t st) {
     constexpr int HM = 16 * MT;
     const size_t smem = split_smem<MT>(p.rank);
@@ -551,11 +553,11 @@ static int split_launch(juno_ctx *c, const SplitParams &p, int n, cudaStream_t s
     {
         std::lock_guard<std::mutex> lk(mu);
         if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(latent_split_kernel<MT, NQ, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(latent_split_kernel<MT, NQ, NP, RANK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             have[c->device & 15] = smem;
         }
     }
-    JUNO_CUDA_TRY(launch_pdl(latent_split_kernel<MT, NQ, NP>, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
+    JUNO_CUDA_TRY(launch_pdl(latent_split_kernel<MT, NQ, NP, RANK>, dim3((unsigned)p.n_splits, (unsigned)((p.heads + HM - 1) / HM), (unsigned)n), dim3(kSpThreads), smem, st, p));
     c->kernel_launches++;
     return JUNO_OK;
 }
@@ -579,6 +581,7 @@ int launch_latent_attn_split(juno_ctx *c, const LatentSplitArgs &a, cudaStream_t
     p.part_ml = a.part_ml;
     ProfScope prof(c, st, PROF_ATTN, 0);
     const int n = a.rows.n;
+    if (a.rank == 512) return a.heads <= 16 ? split_launch<1, 4, 2, 512>(c, p, n, st) : split_launch<2, 4, 2, 512>(c, p, n, st);
     if (a.rank > 512) return split_launch<1, 8, 4>(c, p, n, st);
     if (a.heads <= 16) return a.rank <= 256 ? split_launch<1, 2, 1>(c, p, n, st) : split_launch<1, 4, 2>(c, p, n, st);
     return a.rank <= 256 ? split_launch<2, 2, 1>(c, p, n, st) : split_launch<2, 4, 2>(c, p, n, st);

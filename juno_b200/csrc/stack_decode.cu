@@ -22,7 +22,8 @@ bool stack_fused_ok(const juno_ctx *c, const StackNet *net, const RowSet &rows) 
         if (m.rp() > 1024) return false;
         cols = std::max(cols, std::max(m.qp(), m.heads * std::max(m.dp(), m.vp())));
     }
-    return gemv_rows_chunk(c, cols, 1, 1) > 0 && gemv_rows_chunk(c, net->spec.wp(), 2, 1) > 0;
+    // operands that need more than two passes over the weights: one pass on the row products is faster
+    return 2 * gemv_rows_chunk(c, cols, 1, rows.n) >= rows.n && 2 * gemv_rows_chunk(c, net->spec.wp(), 2, rows.n) >= rows.n;
 }
 
 static GvSeg seg(const StackMat &w, int epi, void *out, int ldo) {
