@@ -331,6 +331,18 @@ def test_generation_in_batches_equals_generation_alone(tmp_path):
     h.release_gpu_resources()
 
 
+def test_generation_from_the_command_line(tmp_path, capsys):
+    from juno_b200 import generate
+    p = Pair(tmp_path, CONFIGS["odd"], 43)
+    prompts = [p.tokens(12, 1), p.tokens(3, 2)]
+    arg = [",".join(map(str, s)) for s in prompts]
+    lines = []
+    for args in (["--ids", arg[0]], ["--ids", arg[0], "--token-by-token"], ["--ids", arg[1]], ["--ids", arg[0], "--ids", arg[1]]):
+        assert generate.main([p.dir, "--steps", "9", "--dtype", "f32", *args]) == 0
+        lines.append(capsys.readouterr().out.split())
+    assert lines[0] == lines[1] and lines[3] == lines[0] + lines[2] and len(lines[0][0].split(",")) == 9
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_trace_replay(tmp_path, dtype):
     from juno_b200 import trace
