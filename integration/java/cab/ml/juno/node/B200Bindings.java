@@ -84,6 +84,10 @@ final class B200Bindings {
 	static final MethodHandle forward = h("juno_forward", fn(ADDRESS, JAVA_INT, ADDRESS, ADDRESS, ADDRESS, ADDRESS, ADDRESS));
 	static final MethodHandle prefill = h("juno_prefill", fn(ADDRESS, ADDRESS, ADDRESS, JAVA_INT, JAVA_INT, ADDRESS, ADDRESS));
 	static final MethodHandle decodeGreedy = h("juno_decode_greedy", fn(ADDRESS, JAVA_INT, ADDRESS, ADDRESS, ADDRESS, JAVA_INT, ADDRESS));
+	/** juno_open_opts: struct_size, max_batch, max_seqs, max_ctx, dtype, max_rows (six 32-bit fields, 24 bytes). */
+	static final MethodHandle modelOpen = h("juno_model_open", fn(ADDRESS, ADDRESS, ADDRESS, ADDRESS));
+	static final MethodHandle modelDescribe = h("juno_model_describe", fn(ADDRESS, ADDRESS));
+	static final MethodHandle prefillLogits = h("juno_prefill_logits", fn(ADDRESS, ADDRESS, ADDRESS, JAVA_INT, JAVA_INT, JAVA_INT, ADDRESS, ADDRESS));
 	static final MethodHandle lastHidden = h("juno_model_last_hidden", fn(ADDRESS, JAVA_INT, ADDRESS));
 
 	private B200Bindings() {
