@@ -17,7 +17,9 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libjuno_b200.so")
 SOURCES = ["context.cu", "gemv.cu", "qgemv.cu", "gemm.cu", "gemm_tc.cu", "attn.cu", "model.cu", "gguf_file.cu",
-           "safetensors_file.cu", "registry.cu", "vosotar.cu", "stack.cu", "stack_decode.cu", "gemv_rows.cu", "rowops.cu", "gemm_rows.cu", "gemm_rows_tc.cu", "latent_attn.cu", "latent_attn_mma.cu"]
+           "safetensors_file.cu", "registry.cu", "stack_loader.cu", "vosotar.cu", "desilorn.cu", "stack.cu", "stack_decode.cu", "gemv_rows.cu",
+           "rowops.cu", "streams.cu", "gemm_rows.cu", "gemm_rows_tc.cu", "latent_attn.cu", "latent_attn_mma.cu", "flash_attn.cu",
+           "grouped_attn.cu"]
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 
 

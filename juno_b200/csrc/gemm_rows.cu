@@ -11,7 +11,7 @@ template <typename T>
 __device__ __forceinline__ void simt_epilogue(const GemmArgs &p, int z, int m, int n, float v) {
     const size_t o = (size_t)m * p.ldo + (size_t)z * p.o_step + n;
     if (p.epi == GE_F32) {
-        static_cast<float *>(p.out)[o] = v;
+        static_cast<float *>(p.out)[o] = p.bias ? v + p.bias[n] : v;
         return;
     }
     if (p.epi == GE_SIGMOID) v = sigmoid_f32(v + p.bias[n]);
@@ -57,12 +57,19 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const GemmArgs p) {
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+            if (p.epi == GE_GEGLU) {  // the value of column n is eight columns on: two threads further
+                const float value = __shfl_down_sync(0xffffffffu, acc[i][j], 2);
+                if (m < p.M && n < p.N && !(n & 8))
+                    static_cast<T *>(p.out)[(size_t)m * p.ldo + (n >> 4) * 8 + (n & 7)] = Num<T>::put(gelu_tanh(acc[i][j]) * value);
+                continue;
+            }
             if (m < p.M && n < p.N) simt_epilogue<T>(p, z, m, n, acc[i][j]);
         }
 }
 
 int launch_gemm_rows(juno_ctx *c, int dt, const GemmArgs &a, unsigned *err, cudaStream_t st) {
-    JUNO_REQUIRE(a.a && a.w && a.out && a.M > 0 && a.N > 0 && a.K > 0 && a.K % 16 == 0 && a.lda % 16 == 0 && a.ldw % 16 == 0 && a.a_step % 16 == 0 && a.groups >= 1,
+    JUNO_REQUIRE(a.a && a.w && a.out && a.M > 0 && a.N > 0 && a.K > 0 && a.K % 16 == 0 && a.lda % 16 == 0 && a.ldw % 16 == 0 && a.a_step % 16 == 0 && a.groups >= 1 &&
+                     (a.epi != GE_GEGLU || (a.N % 16 == 0 && a.groups == 1)),
                  "matrix product: bad arguments (M %d, N %d, K %d)", a.M, a.N, a.K);
     const double es = dt_bytes(dt);
     const double algo = a.groups * ((double)a.M * a.K + (double)a.N * a.K) * es + (double)a.groups * a.M * a.N * (a.epi == GE_F32 ? 4.0 : es);

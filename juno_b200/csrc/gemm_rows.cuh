@@ -5,12 +5,13 @@
 namespace juno {
 
 enum GemmEpi {
-    GE_F32 = 0,      // FP32 result
+    GE_F32 = 0,      // acc (+ bias[n] when there is one), FP32
     GE_OP,           // operand type
     GE_SIGMOID,      // sigmoid(acc + bias[n]), operand type
     GE_RELU2,        // max(acc, 0)^2, operand type
     GE_MUL,          // acc * aux[m][n] (operand type), operand type
     GE_GROUP_GATE,   // acc * sigmoid(gate[m][group]) (FP32), operand type
+    GE_GEGLU,        // columns in tiles of 8 gates and the 8 values they gate: gelu_tanh(gate) * value, operand type, half as many columns
 };
 
 // `groups` > 1: a block-diagonal product (one block per attention head): group z multiplies columns a_step*z.. of `a` with rows

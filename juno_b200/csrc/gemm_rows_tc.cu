@@ -84,6 +84,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
 }
 
 __device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float fast_geglu(float z, float v) { return z * v * fast_sigmoid(1.5957691216057308f * fmaf(0.044715f * z * z, z, z)); }
 
 // 32 columns of one output row.  nv = columns that exist (0..32).
 template <int EPI>
@@ -91,7 +92,15 @@ __device__ __forceinline__ void store_row(const GemmArgs &g, int z, int m, int n
     const size_t o = (size_t)m * g.ldo + (size_t)z * g.o_step + n;
     if (EPI == GE_F32) {
         float *out = static_cast<float *>(g.out) + o;
-        if (nv == 32 && (g.ldo & 3) == 0 && (g.o_step & 3) == 0) {
+        if (g.bias) {  // nv is a multiple of 16 then
+#pragma unroll
+            for (int j = 0; j < 32; j += 4) {
+                if (j >= nv) break;
+                const float4 b = *reinterpret_cast<const float4 *>(g.bias + n + j);
+                *reinterpret_cast<float4 *>(out + j) =
+                    make_float4(__uint_as_float(r[j]) + b.x, __uint_as_float(r[j + 1]) + b.y, __uint_as_float(r[j + 2]) + b.z, __uint_as_float(r[j + 3]) + b.w);
+            }
+        } else if (nv == 32 && (g.ldo & 3) == 0 && (g.o_step & 3) == 0) {
 #pragma unroll
             for (int j = 0; j < 32; j += 4)
                 *reinterpret_cast<float4 *>(out + j) = make_float4(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), __uint_as_float(r[j + 2]), __uint_as_float(r[j + 3]));
@@ -99,6 +108,19 @@ __device__ __forceinline__ void store_row(const GemmArgs &g, int z, int m, int n
 #pragma unroll
             for (int j = 0; j < 32; j++)
                 if (j < nv) out[j] = __uint_as_float(r[j]);
+        }
+        return;
+    }
+    if (EPI == GE_GEGLU) {
+        bf16 *act = static_cast<bf16 *>(g.out) + (size_t)m * g.ldo + (n >> 1);
+#pragma unroll
+        for (int j = 0; j < 32; j += 16) {
+            if (j >= nv) break;
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; e++) v[e] = fast_geglu(__uint_as_float(r[j + e]), __uint_as_float(r[j + 8 + e]));
+            store4(act + j / 2, make_float4(v[0], v[1], v[2], v[3]));
+            store4(act + j / 2 + 4, make_float4(v[4], v[5], v[6], v[7]));
         }
         return;
     }
@@ -297,6 +319,7 @@ static int gemm_tc_epi(juno_ctx *c, const GemmTcParams &p, cudaStream_t st) {
     case GE_SIGMOID: return gemm_tc_inst<BN, GE_SIGMOID>(c, p, st);
     case GE_RELU2: return gemm_tc_inst<BN, GE_RELU2>(c, p, st);
     case GE_MUL: return gemm_tc_inst<BN, GE_MUL>(c, p, st);
+    case GE_GEGLU: return gemm_tc_inst<BN, GE_GEGLU>(c, p, st);
     default: return gemm_tc_inst<BN, GE_GROUP_GATE>(c, p, st);
     }
 }

@@ -75,7 +75,7 @@ struct GvWalk {
 template <int PRO, int COLS>
 __global__ void __launch_bounds__(kGvThreads, 1) gemv_rows_kernel(const __grid_constant__ GvParams p) {
     extern __shared__ __align__(128) uint8_t sm[];
-    __shared__ float red_s[33];
+    __shared__ float red_s[33], coef_s[kMaxStreams + 1];
     const GvArgs &a = p.a;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     float *red = reinterpret_cast<float *>(sm);           // [2][kGvRedFloats]
@@ -119,6 +119,13 @@ __global__ void __launch_bounds__(kGvThreads, 1) gemv_rows_kernel(const __grid_c
     for (int d = 0; d < kGvDepth; d++)
         if (!walk.done(pc)) fetch(w[d]);
 
+    if (PRO == GVP_STREAMS && tid <= a.streams) {  // the sublayer's input as a sum over the old streams and the pending result
+        float v = tid < a.streams && !a.z ? a.hc_in[tid] : 0.f;
+        if (a.z)
+            for (int t = 0; t < a.streams; t++) v = fmaf(tid < a.streams ? a.hc_mix[tid * a.streams + t] : a.hc_out[t], a.hc_in[t], v);
+        coef_s[tid] = v;
+    }
+
     pdl_wait();
     pdl_launch_dependents();
 
@@ -144,6 +151,72 @@ __global__ void __launch_bounds__(kGvThreads, 1) gemv_rows_kernel(const __grid_c
                 const float r = 1.f / sqrtf(block_sum(sk, red_s) / (float)a.kv_rank + a.eps);
                 bf16 *dst = latent_row(a.plane, a.table + (size_t)a.slots[b] * a.max_pages, a.page_width, a.positions[b]);
                 for (int i = tid; i < a.page_width; i += kGvThreads) dst[i] = __float2bfloat16_rn(i < a.kv_rank ? c[i] * r * a.wkv[i] : 0.f);
+            }
+        }
+    } else if (PRO == GVP_STREAMS) {
+        __syncthreads();
+        const int S = a.streams;
+        float4 nw[COLS];
+#pragma unroll
+        for (int i = 0; i < COLS; i++) {
+            const int col = (i * kGvThreads + tid) * 4;
+            if (col < a.K) nw[i] = load4(a.norm_w + col);
+        }
+        for (int b = 0; b < a.n; b++) {
+            const float *x = a.x + (size_t)b * S * a.K, *z = a.z ? a.z + (size_t)b * a.K : nullptr;
+            float4 u[COLS];
+            float sx = 0.f;
+#pragma unroll
+            for (int i = 0; i < COLS; i++) {
+                const int col = (i * kGvThreads + tid) * 4;
+                u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (col >= a.K) continue;
+                if (z) {
+                    const float4 y = load4(z + col);
+                    const float c = coef_s[S];
+                    u[i] = make_float4(c * y.x, c * y.y, c * y.z, c * y.w);
+                }
+#pragma unroll 4
+                for (int s = 0; s < S; s++) {
+                    const float4 v = load4(x + (size_t)s * a.K + col);
+                    const float c = coef_s[s];
+                    u[i].x = fmaf(c, v.x, u[i].x);
+                    u[i].y = fmaf(c, v.y, u[i].y);
+                    u[i].z = fmaf(c, v.z, u[i].z);
+                    u[i].w = fmaf(c, v.w, u[i].w);
+                }
+                sx += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
+            }
+            const float k = 1.f / sqrtf(block_sum(sx, red_s) / (float)a.width + a.eps);
+#pragma unroll
+            for (int i = 0; i < COLS; i++) {
+                const int col = (i * kGvThreads + tid) * 4;
+                if (col < a.K)
+                    store4(reinterpret_cast<bf16 *>(ops + (size_t)b * p.pitch) + col,
+                           make_float4(u[i].x * k * nw[i].x, u[i].y * k * nw[i].y, u[i].z * k * nw[i].z, u[i].w * k * nw[i].w));
+            }
+        }
+        if (a.z) {  // every CTA stores its share of the new streams
+            const int groups = a.K >> 2, total = a.n * groups, per = (total + (int)gridDim.x - 1) / (int)gridDim.x;
+            const int end = min(total, ((int)blockIdx.x + 1) * per);
+            for (int e = (int)blockIdx.x * per + tid; e < end; e += kGvThreads) {
+                const int b = e / groups, col = (e - b * groups) * 4;
+                const float *x = a.x + (size_t)b * S * a.K + col;
+                const float4 y = load4(a.z + (size_t)b * a.K + col);
+                for (int t = 0; t < S; t++) {
+                    const float o = a.hc_out[t];
+                    float4 v = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll 4
+                    for (int s = 0; s < S; s++) {
+                        const float4 w4 = load4(x + (size_t)s * a.K);
+                        const float m = a.hc_mix[s * S + t];
+                        v.x = fmaf(m, w4.x, v.x);
+                        v.y = fmaf(m, w4.y, v.y);
+                        v.z = fmaf(m, w4.z, v.z);
+                        v.w = fmaf(m, w4.w, v.w);
+                    }
+                    store4(a.x_store + ((size_t)b * S + t) * a.K + col, v);
+                }
             }
         }
     } else {
@@ -305,18 +378,22 @@ __global__ void __launch_bounds__(kGvThreads, 1) gemv_rows_kernel(const __grid_c
             if (b >= a.n) continue;
             int w_lo, w_hi;
             qsplit_row_tile_warps(lt, p.nkb, T, w_lo, w_hi);
-            float v = 0.f;
-            for (int x = w_lo; x <= w_hi; x++) {
-                int e0, e1;
-                qsplit_warp(x, T, e0, e1);
-                if (e0 < e1) v += cred[(x * 2 + (e0 / p.nkb == lt ? 0 : 1)) * 128 + r * 8 + b];
-            }
+            auto total = [&](int rr) {
+                float v = 0.f;
+                for (int x = w_lo; x <= w_hi; x++) {
+                    int e0, e1;
+                    qsplit_warp(x, T, e0, e1);
+                    if (e0 < e1) v += cred[(x * 2 + (e0 / p.nkb == lt ? 0 : 1)) * 128 + rr * 8 + b];
+                }
+                return v;
+            };
+            const float v = total(r);
             const int rt = lo + lt, si = seg_of(rt), row = (rt - p.seg_rt[si]) * 16 + r;
             const GvSeg &sg = a.seg[si];
             if (sg.n_store && row >= sg.n_store) continue;
             const size_t idx = (size_t)b * sg.ldo + row;
             switch (sg.epi) {
-            case GVE_F32: static_cast<float *>(sg.out)[idx] = v; break;
+            case GVE_F32: static_cast<float *>(sg.out)[idx] = sg.bias ? v + sg.bias[row] : v; break;
             case GVE_OP: static_cast<bf16 *>(sg.out)[idx] = __float2bfloat16_rn(v); break;
             case GVE_SIGMOID: static_cast<float *>(sg.out)[idx] = sigmoid_f32(v + sg.bias[row]); break;
             case GVE_RELU2: {
@@ -324,6 +401,9 @@ __global__ void __launch_bounds__(kGvThreads, 1) gemv_rows_kernel(const __grid_c
                 static_cast<bf16 *>(sg.out)[idx] = __float2bfloat16_rn(y * y);
                 break;
             }
+            case GVE_GEGLU:
+                if (r < 8) static_cast<bf16 *>(sg.out)[(size_t)b * sg.ldo + (row >> 4) * 8 + r] = __float2bfloat16_rn(gelu_tanh(v) * total(r + 8));
+                break;
             default: static_cast<float *>(sg.out)[idx] = v * sg.aux[(size_t)b * sg.ldaux + row];
             }
         }
@@ -378,12 +458,16 @@ static int launch_one(juno_ctx *c, const GvArgs &a, cudaStream_t st) {
     ProfScope prof(c, st, PROF_GEMV_ROWS, bytes);
     if (a.prologue == GVP_COPY) return launch_inst<GVP_COPY, 1>(c, p, smem, st);
     if (a.prologue == GVP_LATENT) return launch_inst<GVP_LATENT, 1>(c, p, smem, st);
+    if (a.prologue == GVP_STREAMS) return a.K <= 4096 ? launch_inst<GVP_STREAMS, 2>(c, p, smem, st) : launch_inst<GVP_STREAMS, 4>(c, p, smem, st);
     return a.K <= 4096 ? launch_inst<GVP_RESIDUAL, 2>(c, p, smem, st) : launch_inst<GVP_RESIDUAL, 4>(c, p, smem, st);
 }
 
 int launch_gemv_rows(juno_ctx *c, const GvArgs &a, cudaStream_t st) {
     JUNO_REQUIRE(a.n >= 1 && a.n <= kGvMaxSeqs && a.K > 0 && a.K % 16 == 0 && a.nseg >= 1 && a.nseg <= 3, "decode product: bad arguments (n %d, K %d)", a.n, a.K);
     JUNO_REQUIRE(a.prologue != GVP_RESIDUAL || (a.K <= kGvMaxWidth && a.width <= a.K), "decode product: a residual row of %d is too wide", a.K);
+    JUNO_REQUIRE(a.prologue != GVP_STREAMS || (a.K <= kGvMaxWidth && a.width <= a.K && a.streams >= 1 && a.streams <= kMaxStreams && a.x && a.hc_in && a.norm_w &&
+                                               (!a.z || (a.hc_mix && a.hc_out && a.x_store && a.x_store != a.x))),
+                 "decode product: bad streams");
     JUNO_REQUIRE(a.group_rows % 16 == 0, "decode product: groups of %d rows", a.group_rows);
     for (int s = 0; s < a.nseg; s++) JUNO_REQUIRE(a.seg[s].rows > 0 && a.seg[s].rows % 16 == 0 && a.seg[s].w && a.seg[s].out, "decode product: bad segment %d", s);
     const int n_op = a.prologue == GVP_RESIDUAL && a.conv_w ? 2 : 1;
@@ -393,15 +477,16 @@ int launch_gemv_rows(juno_ctx *c, const GvArgs &a, cudaStream_t st) {
         GvArgs t = a;
         t.n = std::min(step, a.n - b);
         if (t.in) t.in += (size_t)b * t.ld_in;
-        if (t.x) t.x += (size_t)b * t.K;
+        const size_t x_row = (size_t)t.K * std::max(t.streams, 1);
+        if (t.x) t.x += b * x_row;
         if (t.z) t.z += (size_t)b * t.K;
-        if (t.x_store) t.x_store += (size_t)b * t.K;
+        if (t.x_store) t.x_store += b * x_row;
         if (t.u) t.u += (size_t)b * t.ldu;
         if (t.positions) t.positions += b;
         if (t.slots) t.slots += b;
         for (int s = 0; s < t.nseg; s++) {
             GvSeg &g = t.seg[s];
-            const size_t es = g.epi == GVE_OP || g.epi == GVE_RELU2 ? 2 : 4;
+            const size_t es = g.epi == GVE_OP || g.epi == GVE_RELU2 || g.epi == GVE_GEGLU ? 2 : 4;
             g.out = static_cast<uint8_t *>(g.out) + (size_t)b * g.ldo * es;
             if (g.aux) g.aux += (size_t)b * g.ldaux;
         }

@@ -1,15 +1,22 @@
 // Fused BF16 matrix-vector products of a decode step (one to eight sequences): the operand is built from FP32 rows inside the
-// consuming product - residual sum, norms, short convolution, latent norm - and the weights stream past it once.
+// consuming product - residual sum or residual streams, norms, short convolution, latent norm - and the weights stream past it once.
 #pragma once
-#include "rowops.cuh"
+#include "streams.cuh"
 
 namespace juno {
 
 constexpr int kGvMaxSeqs = 8;
 constexpr int kGvMaxWidth = 8192;  // widest residual row the fused residual prologue takes
 
-enum GvPrologue { GVP_COPY = 0, GVP_RESIDUAL, GVP_LATENT };
-enum GvEpi { GVE_F32 = 0, GVE_OP, GVE_SIGMOID /* sigmoid(v + bias), FP32 */, GVE_RELU2 /* BF16 */, GVE_MUL /* v * aux, FP32 */ };
+enum GvPrologue { GVP_COPY = 0, GVP_RESIDUAL, GVP_LATENT, GVP_STREAMS };
+enum GvEpi {
+    GVE_F32 = 0,  // v (+ bias when there is one), FP32
+    GVE_OP,
+    GVE_SIGMOID,  // sigmoid(v + bias), FP32
+    GVE_RELU2,    // BF16
+    GVE_MUL,      // v * aux, FP32
+    GVE_GEGLU,    // rows in tiles of 8 gates and the 8 values they gate: gelu_tanh(gate) * value, BF16, half as many columns
+};
 
 struct GvSeg {
     const __nv_bfloat16 *w = nullptr;  // [rows][ldw], ldw = the launch's K padded to 16
@@ -42,6 +49,10 @@ struct GvArgs {
     float *state = nullptr;                 // this layer's state rows of slot 0
     size_t slot_stride = 0;
     int ring_mask = 0;
+    // GVP_STREAMS (see streams.cuh): x [n][streams][K]; the pending result z [n][K] is mixed in with hc_mix and hc_out,
+    // operand = rms(sum_s hc_in[s] x_s) * norm_w; the new streams go to x_store
+    int streams = 0;
+    const float *hc_mix = nullptr, *hc_out = nullptr, *hc_in = nullptr, *norm_w = nullptr;
     // GVP_LATENT: u [n][ldu]: operand = rms(u[0..q_rank)) * wq; u[kv_col..+kv_rank) is normed with wkv and appended to the pages
     const float *u = nullptr, *wq = nullptr, *wkv = nullptr;
     int ldu = 0, q_rank = 0, kv_col = 0, kv_rank = 0, page_width = 0, max_pages = 0;

@@ -46,20 +46,6 @@ struct LatentMergeArgs {
 };
 int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st);
 
-// BF16, many rows of one sequence: keys and values expanded from the latent once per pass, causal flash attention over them.
-// kv [positions][ldkv]: keys of all heads (heads * dim), then values (heads * vdim); row r is position pos0 + r.
-struct FlashArgs {
-    int n, pos0, heads, dim, vdim;  // padded sizes
-    float scale;
-    const void *q;      // [n][heads * dim]
-    const void *kv;
-    int ldkv;
-    const float *gate;  // [n][ld_gate], one per head (null: none)
-    int ld_gate;
-    void *out;          // [n][heads * vdim]
-};
-constexpr int kFlashMaxDim = 256;
-int launch_flash_prefill(juno_ctx *c, const FlashArgs &a, cudaStream_t st);
 // out[j][rank] = the latent of position j of the sequence in `slot_of` (device, one word), j < len
 int launch_latent_gather(juno_ctx *c, const juno_kvpool *pool, int layer, const int32_t *slot_of, int len, void *out, cudaStream_t st);
 

@@ -1,5 +1,4 @@
-// BF16 attention over latent pages on the tensor cores: the split kernel of decode steps with its merge, and causal flash
-// attention over expanded keys and values for prompts (see latent_attn.cuh).
+// BF16 attention over latent pages on the tensor cores: the split kernel of decode steps with its merge (see latent_attn.cuh).
 #include <algorithm>
 #include <mutex>
 
@@ -9,7 +8,6 @@
 namespace juno {
 
 using bf16 = __nv_bfloat16;
-constexpr float kLog2e = 1.4426950408889634f;
 
 // ───────────────────────────── decode: splits of the context ──────────────────────────────
 // A CTA (sixteen warps, one per SM) takes a group of 16 * MT heads of one row and a range of positions, 32 at a time.  Scores:
@@ -27,12 +25,6 @@ struct SplitParams {
     const bf16 *q;
     float *part_o, *part_ml;
 };
-
-__device__ __forceinline__ float ex2(float v) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
-    return r;
-}
 
 __device__ __forceinline__ float warp_max(float v) {
     float r;
@@ -331,183 +323,7 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const Merge
     }
 }
 
-// ───────────────────────────── prompts: causal flash attention ────────────────────────────
-// 128 query rows of one head per CTA, four warps of MT 16-row tiles; 64 keys per step, keys and values double-buffered.
-constexpr int kFlKeys = 64, kFlThreads = 128;
-struct FlashParams {
-    FlashArgs a;
-    float scale_log2;
-};
-template <int D, int MT>  // D: most dimensions per head; MT: 16-row tiles per warp
-__global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_kernel(const FlashParams p) {
-    extern __shared__ __align__(16) uint8_t sm[];
-    constexpr int BR = 64 * MT, NK = D / 16, NV = D / 16;
-    const FlashArgs &a = p.a;
-    const int dp = a.dim, vp = a.vdim, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
-    bf16 *qs = reinterpret_cast<bf16 *>(sm);
-    bf16 *ks = qs + BR * kp;                 // [2][64][kp]
-    bf16 *vs = ks + 2 * kFlKeys * kp;        // [2][64][vpitch]
-    const int h = blockIdx.x, r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * BR;  // long rows first
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const bf16 *q = static_cast<const bf16 *>(a.q) + (size_t)h * dp;
-    const bf16 *kv = static_cast<const bf16 *>(a.kv);
-    const int ldq = a.heads * dp, rows = min(BR, a.n - r0), len = a.pos0 + r0 + rows;  // keys any row of the tile sees
-    const int kc = dp >> 3, vc = vp >> 3;
-    // this thread's first (row, 16-byte piece) of a tile and the step to its next, for keys and values
-    const int kr0 = tid / kc, kch0 = tid - kr0 * kc, krs = kFlThreads / kc, kcs = kFlThreads - krs * kc;
-    const int vr0 = tid / vc, vch0 = tid - vr0 * vc, vrs = kFlThreads / vc, vcs = kFlThreads - vrs * vc;
-    auto load_rows = [&](const bf16 *src, uint32_t dst, int pitch, int j, int r, int ch, int rs, int chs, int nch) {
-        while (r < kFlKeys) {
-            const bool ok = j + r < len;
-            cp16(dst + (uint32_t)(r * pitch + ch * 8) * 2, src + (size_t)(ok ? j + r : 0) * a.ldkv + ch * 8, ok);
-            ch += chs;
-            r += rs;
-            if (ch >= nch) {
-                ch -= nch;
-                r++;
-            }
-        }
-    };
-    auto load_kv = [&](int j, int buf) {
-        load_rows(kv + h * dp, smem_addr(ks + (size_t)buf * kFlKeys * kp), kp, j, kr0, kch0, krs, kcs, kc);
-        load_rows(kv + a.heads * dp + h * vp, smem_addr(vs + (size_t)buf * kFlKeys * vpitch), vpitch, j, vr0, vch0, vrs, vcs, vc);
-        cp_commit();
-    };
-    for (int i = tid; i < BR * kc; i += kFlThreads) {
-        const int r = i / kc, ch = i - r * kc;
-        const bool ok = r < rows;
-        cp16(smem_addr(qs + r * kp + ch * 8), q + (size_t)(ok ? r0 + r : r0) * ldq + ch * 8, ok);
-    }
-    load_kv(0, 0);
-    const int lr = lane & 15, lc = (lane >> 4) * 8, br = (lane & 7) + (lane >> 4) * 8, bc = ((lane >> 3) & 1) * 8;
-    const int g = lane >> 2, t = lane & 3, wrow = warp * 16 * MT;
-    float o[MT][NV][2][4], mx[MT][2], ls[MT][2];
-#pragma unroll
-    for (int m = 0; m < MT; m++) {
-        mx[m][0] = mx[m][1] = -INFINITY;
-        ls[m][0] = ls[m][1] = 0.f;
-#pragma unroll
-        for (int i = 0; i < NV; i++)
-#pragma unroll
-            for (int k = 0; k < 2; k++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) o[m][i][k][e] = 0.f;
-    }
-    int buf = 0;
-    for (int j = 0; j < len; j += kFlKeys, buf ^= 1) {
-        cp_wait<0>();
-        __syncthreads();
-        if (j + kFlKeys < len) load_kv(j + kFlKeys, buf ^ 1);
-        if (j > a.pos0 + r0 + wrow + 16 * MT - 1) continue;  // every key of the tile lies behind this warp's rows
-        const bf16 *kt = ks + (size_t)buf * kFlKeys * kp, *vt = vs + (size_t)buf * kFlKeys * vpitch;
-        float s[MT][kFlKeys / 8][4];
-#pragma unroll
-        for (int m = 0; m < MT; m++)
-#pragma unroll
-            for (int i = 0; i < kFlKeys / 8; i++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) s[m][i][e] = 0.f;
-#pragma unroll
-        for (int k = 0; k < NK; k++) {
-            if (k < nk) {
-                uint32_t qa[MT][4];
-#pragma unroll
-                for (int m = 0; m < MT; m++) ldsm4(qa[m], smem_addr(qs + (wrow + m * 16 + lr) * kp + k * 16 + lc));
-#pragma unroll
-                for (int i = 0; i < kFlKeys / 16; i++) {
-                    uint32_t b[4];
-                    ldsm4(b, smem_addr(kt + (i * 16 + br) * kp + k * 16 + bc));
-#pragma unroll
-                    for (int m = 0; m < MT; m++) {
-                        mma16816(s[m][2 * i], qa[m], b[0], b[1]);
-                        mma16816(s[m][2 * i + 1], qa[m], b[2], b[3]);
-                    }
-                }
-            }
-        }
-        uint32_t pa[MT][kFlKeys / 16][4];
-#pragma unroll
-        for (int m = 0; m < MT; m++) {
-#pragma unroll
-            for (int e2 = 0; e2 < 2; e2++) {  // rows g and g + 8
-                const int pos = a.pos0 + r0 + wrow + m * 16 + g + e2 * 8;
-                float mv = mx[m][e2];
-                if (j + kFlKeys - 1 > pos) {
-#pragma unroll
-                    for (int i = 0; i < kFlKeys / 8; i++)
-#pragma unroll
-                        for (int e = 0; e < 2; e++)
-                            if (j + i * 8 + 2 * t + e > pos) s[m][i][e2 * 2 + e] = -INFINITY;
-                }
-#pragma unroll
-                for (int i = 0; i < kFlKeys / 8; i++) mv = fmaxf(mv, fmaxf(s[m][i][e2 * 2], s[m][i][e2 * 2 + 1]));
-                mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 1));
-                mv = fmaxf(mv, __shfl_xor_sync(0xffffffffu, mv, 2));
-                const float base = mv == -INFINITY ? 0.f : mv * p.scale_log2;
-                const float f = ex2(mx[m][e2] * p.scale_log2 - base);
-                mx[m][e2] = mv;
-                float sum = 0.f;
-#pragma unroll
-                for (int i = 0; i < kFlKeys / 8; i++)
-#pragma unroll
-                    for (int e = 0; e < 2; e++) {
-                        const float v = ex2(fmaf(s[m][i][e2 * 2 + e], p.scale_log2, -base));
-                        s[m][i][e2 * 2 + e] = v;
-                        sum += v;
-                    }
-                ls[m][e2] = ls[m][e2] * f + sum;
-#pragma unroll
-                for (int i = 0; i < NV; i++)
-#pragma unroll
-                    for (int k = 0; k < 2; k++) {
-                        o[m][i][k][e2 * 2] *= f;
-                        o[m][i][k][e2 * 2 + 1] *= f;
-                    }
-            }
-#pragma unroll
-            for (int i = 0; i < kFlKeys / 16; i++) {
-                pa[m][i][0] = pack_bf16(s[m][2 * i][0], s[m][2 * i][1]);
-                pa[m][i][1] = pack_bf16(s[m][2 * i][2], s[m][2 * i][3]);
-                pa[m][i][2] = pack_bf16(s[m][2 * i + 1][0], s[m][2 * i + 1][1]);
-                pa[m][i][3] = pack_bf16(s[m][2 * i + 1][2], s[m][2 * i + 1][3]);
-            }
-        }
-#pragma unroll
-        for (int kk = 0; kk < kFlKeys / 16; kk++)
-#pragma unroll
-            for (int i = 0; i < NV; i++) {
-                if (i < nv) {
-                    uint32_t b[4];
-                    ldsm4_trans(b, smem_addr(vt + (kk * 16 + lr) * vpitch + i * 16 + lc));
-#pragma unroll
-                    for (int m = 0; m < MT; m++) {
-                        mma16816(o[m][i][0], pa[m][kk], b[0], b[1]);
-                        mma16816(o[m][i][1], pa[m][kk], b[2], b[3]);
-                    }
-                }
-            }
-    }
-#pragma unroll
-    for (int m = 0; m < MT; m++)
-#pragma unroll
-        for (int e2 = 0; e2 < 2; e2++) {
-            float l = ls[m][e2];
-            l += __shfl_xor_sync(0xffffffffu, l, 1);
-            l += __shfl_xor_sync(0xffffffffu, l, 2);
-            const int r = wrow + m * 16 + g + e2 * 8;
-            if (r >= rows) continue;
-            float f = 1.f / l;
-            if (a.gate) f *= sigmoid_f32(a.gate[(size_t)(r0 + r) * a.ld_gate + h]);
-            bf16 *out = static_cast<bf16 *>(a.out) + (size_t)(r0 + r) * a.heads * vp + h * vp;
-#pragma unroll
-            for (int i = 0; i < NV; i++)
-                if (i < nv)
-#pragma unroll
-                    for (int k = 0; k < 2; k++)
-                        *reinterpret_cast<uint32_t *>(out + i * 16 + k * 8 + 2 * t) = pack_bf16(o[m][i][k][e2 * 2] * f, o[m][i][k][e2 * 2 + 1] * f);
-        }
-}
-
+// ───────────────────────────── latents of a sequence, side by side ────────────────────────
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint8_t *plane, const int32_t *table, int max_pages, const int32_t *slot_of, int len,
                                                             int row_bytes, uint8_t *out) {
     const int per = row_bytes >> 4;
@@ -601,39 +417,6 @@ int launch_latent_merge(juno_ctx *c, const LatentMergeArgs &a, cudaStream_t st) 
     JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;
-}
-
-template <int D, int MT>
-static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
-    constexpr int BR = 64 * MT;
-    const size_t smem = ((size_t)(BR + 2 * kFlKeys) * (p.a.dim + 8) + (size_t)2 * kFlKeys * (p.a.vdim + 8)) * 2;
-    static std::mutex mu;
-    static size_t have[16] = {0};
-    {
-        std::lock_guard<std::mutex> lk(mu);
-        if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(flash_prefill_kernel<D, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            have[c->device & 15] = smem;
-        }
-    }
-    flash_prefill_kernel<D, MT><<<dim3((unsigned)p.a.heads, (unsigned)((p.a.n + BR - 1) / BR)), kFlThreads, smem, st>>>(p);
-    JUNO_CUDA_TRY(cudaGetLastError());
-    c->kernel_launches++;
-    return JUNO_OK;
-}
-
-int launch_flash_prefill(juno_ctx *c, const FlashArgs &a, cudaStream_t st) {
-    JUNO_REQUIRE(a.n > 0 && a.pos0 >= 0 && a.heads > 0 && a.dim % 16 == 0 && a.vdim % 16 == 0 && a.dim <= kFlashMaxDim && a.vdim <= kFlashMaxDim && a.ldkv % 8 == 0,
-                 "prompt attention: bad arguments (dim %d, vdim %d)", a.dim, a.vdim);
-    FlashParams p;
-    p.a = a;
-    p.scale_log2 = a.scale * kLog2e;
-    const double pairs = (double)a.n * a.pos0 + (double)a.n * (a.n + 1) / 2;
-    ProfScope prof(c, st, PROF_ATTN, pairs * 2);
-    const int d = std::max(a.dim, a.vdim);
-    if (d <= 64) return flash_launch<64, 2>(c, p, st);
-    if (d <= 128) return flash_launch<128, 2>(c, p, st);
-    return flash_launch<256, 1>(c, p, st);
 }
 
 int launch_latent_gather(juno_ctx *c, const juno_kvpool *pool, int layer, const int32_t *slot_of, int len, void *out, cudaStream_t st) {

@@ -28,6 +28,12 @@ template <int N>
 __device__ __forceinline__ void cp_wait() {
     asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float ex2(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t *>(&v);

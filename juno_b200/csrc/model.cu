@@ -685,7 +685,7 @@ int model_from_stack(juno_ctx *c, StackNet *net, const char *architecture, const
     m->use_graphs = !(ng && *ng == '1');
     auto build = [&]() -> int {
         std::vector<int> widths;
-        for (const StackLayerSpec &L : s.layers) widths.push_back(L.mix.rp());
+        for (const StackLayerSpec &L : s.layers) widths.push_back(L.page_width());
         const int pages_per_seq = (o.max_ctx + kPageTokens - 1) / kPageTokens;
         const long long pages = (long long)o.max_seqs * pages_per_seq;
         JUNO_REQUIRE(pages < (1ll << 31), "latent pool too large");
@@ -695,7 +695,7 @@ int model_from_stack(juno_ctx *c, StackNet *net, const char *architecture, const
             }
         JUNO_TRY(kvpool_create_latent(c, widths, (int)pages, net->dt == DT_F32 ? 1 : 2, o.max_seqs, pages_per_seq, ring, s.wp(), s.taps, &m->pool));
         m->pool->owned_by_model = 1;
-        JUNO_TRY(stack_alloc(c, net, o.max_batch, m->step_cap, m->logit_cap));
+        JUNO_TRY(stack_alloc(c, net, o.max_batch, m->step_cap, m->logit_cap, o.max_ctx));
         JUNO_TRY(dev_alloc((void **)&m->logits_loc, (size_t)m->logit_cap * s.vocab * 4));
         return alloc_step_buffers(m);
     };
@@ -1563,7 +1563,8 @@ int juno_model_last_hidden(juno_model *m, int32_t n, float *hidden_host) {
     juno_ctx *c = m->ctx;
     std::lock_guard<std::recursive_mutex> lk(c->mu);
     DeviceGuard g(c->device);
-    const float *x = m->stack ? stack_residual(m->stack) : m->x[m->last_x];
+    const float *x = m->x[m->last_x];
+    if (m->stack) JUNO_TRY(stack_residual(c, m->stack, n, &x, c->stream));
     const size_t row = (size_t)m->cfg.hidden * 4, pitch = m->stack ? (size_t)m->stack->spec.wp() * 4 : row;
     JUNO_CUDA_TRY(cudaMemcpy2DAsync(hidden_host, row, x, pitch, row, (size_t)n, cudaMemcpyDeviceToHost, c->stream));
     JUNO_CUDA_TRY(cudaStreamSynchronize(c->stream));

@@ -18,6 +18,7 @@ struct Design {
 };
 static const Design kDesigns[] = {
     {"Vosotar", vosotar_spec, vosotar_load},
+    {"Desilorn", desilorn_spec, desilorn_load},
 };
 
 static int open_folder(juno_ctx *c, const std::string &dir, const juno_open_opts &o, juno_model **out) {

@@ -88,6 +88,8 @@ struct Num<__nv_bfloat16> {
     static __device__ __forceinline__ __nv_bfloat16 put(float v) { return __float2bfloat16_rn(v); }
 };
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+// 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), written as z * sigmoid(2 sqrt(2/pi) (...)): no cancellation for z << 0
+__device__ __forceinline__ float gelu_tanh(float z) { return z * sigmoid_f32(1.5957691216057308f * fmaf(0.044715f * z * z, z, z)); }
 
 // Four consecutive elements (16-byte aligned for FP32, 8-byte for BF16).
 __device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }

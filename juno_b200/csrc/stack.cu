@@ -100,10 +100,29 @@ int stack_upload_f32(juno_ctx *c, StackNet *net, const std::vector<float> &v, fl
 // values from the whole context would cost more than it saves.
 constexpr int kAbsorbRows = 48;
 constexpr int kMergeRows = 8;  // rows up to which the value projection is done by the merge of the context splits
-static bool flash_fits(const LatentMixerSpec &m) { return m.dp() <= kFlashMaxDim && m.vp() <= kFlashMaxDim; }
+constexpr int kGroupedFewRows = 16;  // rows of a portion up to which the decode attention is faster than a prompt's
+static bool flash_fits(int dp, int vp) { return dp <= kFlashMaxDim && vp <= kFlashMaxDim; }
 
 // ───────────────────────────── buffers ────────────────────────────────────────────────────
-int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int logit_rows) {
+// (cos, sin) tables, one per distinct rotation.
+static int rotation_tables(juno_ctx *c, StackNet *net, int max_ctx) {
+    const StackSpec &s = net->spec;
+    net->rot.assign(s.layers.size(), nullptr);
+    for (size_t l = 0; l < s.layers.size(); l++) {
+        const GroupedMixerSpec &m = s.layers[l].grouped;
+        if (s.layers[l].mixer != MIX_GROUPED || m.rot_dims == 0) continue;
+        for (size_t k = 0; k < l && !net->rot[l]; k++)
+            if (net->rot[k] && s.layers[k].grouped.rot_dims == m.rot_dims && s.layers[k].grouped.rot_base == m.rot_base) net->rot[l] = net->rot[k];
+        if (net->rot[l]) continue;
+        float2 *t = nullptr;
+        JUNO_TRY(net_alloc(net, (void **)&t, (size_t)max_ctx * (m.rot_dims / 2) * sizeof(float2)));
+        JUNO_TRY(launch_rotation_table(c, max_ctx, m.rot_dims, m.rot_base, t, c->stream));
+        net->rot[l] = t;
+    }
+    return JUNO_OK;
+}
+
+int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int logit_rows, int max_ctx) {
     const StackSpec &s = net->spec;
     const size_t es = dt_bytes(net->dt);
     const int cap = net->cap = std::max(max_batch, max_rows);
@@ -111,37 +130,48 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
     // absorbed queries are kept for few rows only, unless some layer has to take the general kernel
     net->lat_cap = net->dt == DT_BF16 ? std::min(cap, std::max(max_batch, kAbsorbRows)) : cap;
     for (const StackLayerSpec &L : s.layers)
-        if (!flash_fits(L.mix) || L.mix.rp() > kLatentSplitMaxRank) net->lat_cap = cap;
-    const int wp = s.wp();
+        if (L.mixer == MIX_LATENT && (!flash_fits(L.mix.dp(), L.mix.vp()) || L.mix.rp() > kLatentSplitMaxRank)) net->lat_cap = cap;
+    const int wp = s.wp(), streams = std::max(1, s.streams), few = std::min(cap, kGvMaxSeqs);
+    const size_t gated = s.streams ? 0 : 1;  // buffers of the gated, convolved residual
     int ff = 16;
+    bool grouped = false;
     for (const StackLayerSpec &L : s.layers) {
+        ff = std::max(ff, pad16(L.ff));
+        if (L.mixer == MIX_GROUPED) {
+            const GroupedMixerSpec &m = L.grouped;
+            grouped = true;
+            net->ldu = std::max(net->ldu, m.qkv_rows());
+            net->ldq = std::max(net->ldq, m.heads * m.dp());
+            net->ldatt = std::max(net->ldatt, m.heads * m.vp());
+            if (net->dt == DT_BF16 && std::max(m.dp(), m.vp()) <= kGroupedMaxDim) net->part_floats = std::max(net->part_floats, grouped_part_floats(c, m.vp()));
+            continue;
+        }
         const LatentMixerSpec &m = L.mix;
         net->ldu = std::max(net->ldu, m.down_rows());
         net->ldcq = std::max(net->ldcq, m.qp());
         net->ldq = std::max(net->ldq, m.heads * m.dp());
         net->ldlat = std::max(net->ldlat, m.heads * m.rp());
         net->ldatt = std::max(net->ldatt, m.heads * m.vp());
-        ff = std::max(ff, pad16(L.ff));
+        if (net->dt == DT_BF16)
+            for (int n = 1; n <= net->lat_cap; n++) net->part_floats = std::max(net->part_floats, latent_part_floats(c, n, m.heads, m.rp()));
     }
+    for (const StackLayerSpec &L : s.layers)
+        JUNO_REQUIRE((L.mixer == MIX_GROUPED) == (s.streams > 0), "latent attention belongs to the gated residual, grouped attention to residual streams");
     net->ldact = ff;
     net->weight_bytes = (double)net->head.rows * net->head.cols * es;
     for (size_t l = 0; l < s.layers.size(); l++) {
         const StackLayerWeights &L = net->layers[(size_t)s.weights((int)l)];
-        for (const StackMat *m : {&L.down, &L.uq, &L.ukt, &L.o, &L.rg1, &L.rg2, &L.up, &L.mdown}) net->weight_bytes += (double)m->rows * m->cols * es;
-        net->weight_bytes += (double)s.layers[l].mix.heads * s.layers[l].mix.vp() * s.layers[l].mix.rp() * es;  // W_uv
+        for (const StackMat *m : {&L.down, &L.uq, &L.ukt, &L.o, &L.rg1, &L.rg2, &L.up, &L.mdown, &L.qkv, &L.gu}) net->weight_bytes += (double)m->rows * m->cols * es;
+        if (s.layers[l].mixer == MIX_LATENT) net->weight_bytes += (double)s.layers[l].mix.heads * s.layers[l].mix.vp() * s.layers[l].mix.rp() * es;  // W_uv
     }
-    if (net->dt == DT_BF16) {
-        for (const StackLayerSpec &L : s.layers)
-            for (int n = 1; n <= net->lat_cap; n++) net->part_floats = std::max(net->part_floats, latent_part_floats(c, n, L.mix.heads, L.mix.rp()));
-        JUNO_TRY(net_alloc(net, (void **)&net->part_o, net->part_floats * 4));
-    }
+    JUNO_TRY(rotation_tables(c, net, max_ctx));
     const struct { void **p; size_t bytes; } bufs[] = {
-        {(void **)&net->x, (size_t)cap * wp * 4},
+        {(void **)&net->x, (size_t)cap * streams * wp * 4},
         {(void **)&net->u, (size_t)cap * net->ldu * 4},
-        {(void **)&net->row_scale, (size_t)cap * 4},
+        {(void **)&net->row_scale, gated * cap * 4},
         {&net->h, (size_t)cap * wp * es},
-        {&net->hc, (size_t)cap * wp * es},
-        {&net->gate, (size_t)cap * wp * es},
+        {&net->hc, gated * cap * wp * es},
+        {&net->gate, gated * cap * wp * es},
         {&net->z, (size_t)cap * wp * es},
         {&net->cq, (size_t)cap * net->ldcq * es},
         {&net->q, (size_t)cap * net->ldq * es},
@@ -151,9 +181,11 @@ int stack_alloc(juno_ctx *c, StackNet *net, int max_batch, int max_rows, int log
         {&net->act, (size_t)cap * net->ldact * es},
         {&net->fin, (size_t)std::max(logit_rows, 1) * wp * es},
         {(void **)&net->row_idx, (size_t)cap * 4},
-        {(void **)&net->x2, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
-        {(void **)&net->dec_gate, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
-        {(void **)&net->dec_z, (size_t)std::min(cap, kGvMaxSeqs) * wp * 4},
+        {(void **)&net->x2, (size_t)few * streams * wp * 4},
+        {(void **)&net->dec_gate, gated * few * wp * 4},
+        {(void **)&net->dec_z, (size_t)few * wp * 4},
+        {(void **)&net->part_o, net->part_floats * 4},
+        {(void **)&net->counters, grouped ? grouped_counters(c) * 4 : 0},
     };
     for (const auto &b : bufs) {
         JUNO_TRY(net_alloc(net, b.p, b.bytes));
@@ -168,6 +200,7 @@ void stack_free(StackNet *net) {
     for (void *p : net->owned) cudaFree(p);
     if (net->ctx_lat) cudaFree(net->ctx_lat);
     if (net->ctx_kv) cudaFree(net->ctx_kv);
+    if (net->hidden) cudaFree(net->hidden);
     delete net;
 }
 
@@ -188,7 +221,15 @@ void stack_step_done(const juno_ctx *c, StackNet *net, int n) {
     for (const StackLayerSpec &L : net->spec.layers) net->last_x ^= L.ff ? 0 : 1;  // one hand-over per sublayer
 }
 
-const float *stack_residual(const StackNet *net) { return net->last_x ? net->x2 : net->x; }
+int stack_residual(juno_ctx *c, StackNet *net, int n, const float **out, cudaStream_t st) {
+    *out = net->last_x ? net->x2 : net->x;
+    if (net->spec.streams == 0) return JUNO_OK;
+    const int wp = net->spec.wp();
+    JUNO_TRY(ensure_device((void **)&net->hidden, &net->hidden_bytes, (size_t)n * wp * 4));
+    JUNO_TRY(launch_stream_gather(c, net->dt, *out, net->spec.streams, wp, net->spec.width, nullptr, n, nullptr, 0.f, net->hidden, wp, st));
+    *out = net->hidden;
+    return JUNO_OK;
+}
 
 // One split count for all layers of a step (it is part of the captured step's key): the largest any layer's shape asks for
 // that every layer's buffers and kernels take.
@@ -196,6 +237,11 @@ int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bou
     if (net->dt != DT_BF16) return 1;
     int best = 1, most = 1 << 30;
     for (const StackLayerSpec &L : net->spec.layers) {
+        if (L.mixer == MIX_GROUPED) {
+            const GroupedMixerSpec &m = L.grouped;
+            best = std::max(best, grouped_pick_splits(c, n, m.heads, m.kv_heads, std::max(m.dp(), m.vp()), m.span.longest(len_bound)));
+            continue;
+        }
         if (L.mix.rp() > kLatentSplitMaxRank) continue;
         best = std::max(best, latent_pick_splits(c, n, L.mix.heads, L.mix.rp(), len_bound));
         most = std::min<long long>(most, (long long)(net->part_floats / ((size_t)n * L.mix.heads * (L.mix.rp() + 2))));
@@ -204,16 +250,77 @@ int stack_pick_splits(const juno_ctx *c, const StackNet *net, int n, int len_bou
 }
 
 // ───────────────────────────── attention of one layer ─────────────────────────────────────
+GroupedAttnArgs grouped_attn_args(const StackNet *net, const StackLayerWeights &L, const juno_kvpool *pool, int layer, const RowSet &rows) {
+    const GroupedMixerSpec &m = net->spec.layers[(size_t)layer].grouped;
+    GroupedAttnArgs a;
+    a.pool = pool;
+    a.layer = layer;
+    a.rows = rows;
+    a.heads = m.heads;
+    a.kv_heads = m.kv_heads;
+    a.dim = m.dim;
+    a.dp = m.dp();
+    a.vp = m.vp();
+    a.scale = m.scale;
+    a.span = m.span;
+    a.slopes = L.slopes;
+    a.sinks = L.sinks;
+    a.u = net->u;
+    a.ldu = m.qkv_rows();
+    a.q_norm = L.q_norm;
+    a.k_norm = L.k_norm;
+    a.eps = net->spec.eps;
+    a.rot = net->rot[(size_t)layer];
+    a.rot_dims = m.rot_dims;
+    a.temp_coef = m.temp_coef;
+    a.temp_every = m.temp_every;
+    a.q = net->q;
+    a.out = net->att;
+    return a;
+}
+int grouped_layer_splits(const juno_ctx *c, const GroupedMixerSpec &m, int n, int n_splits) {
+    return std::min(n_splits, grouped_pick_splits(c, n, m.heads, m.kv_heads, std::max(m.dp(), m.vp()), m.span.longest(1 << 30)));
+}
+
+// u -> att over the layer's pages, this pass's positions appended.
+static int grouped_attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, const juno_kvpool *pool, int layer, const RowSet &rows, int n_splits, int len_bound,
+                             cudaStream_t st) {
+    const GroupedMixerSpec &m = net->spec.layers[(size_t)layer].grouped;
+    const GroupedAttnArgs a = grouped_attn_args(net, L, pool, layer, rows);
+    const int d = std::max(a.dp, a.vp);
+    JUNO_TRY(launch_grouped_prep(c, net->dt, a, st));
+    if (net->dt == DT_F32 || d > kGroupedMaxDim) return launch_grouped_simt(c, net->dt, a, st);
+    if (!rows.one_seq || rows.n <= kGroupedFewRows)
+        return launch_grouped_split(c, a, grouped_layer_splits(c, m, rows.n, n_splits), false, net->part_o, net->part_floats, net->counters, st);
+    FlashArgs f;
+    f.n = rows.n;
+    f.pos0 = len_bound - rows.n;
+    f.heads = a.heads;
+    f.dim = a.dp;
+    f.vdim = a.vp;
+    f.scale = a.scale;
+    f.q = a.q;
+    f.out = a.out;
+    f.kv_heads = a.kv_heads;
+    f.pool = pool;
+    f.layer = layer;
+    f.slot = rows.slots;
+    f.span = a.span;
+    f.slopes = a.slopes;
+    f.sinks = a.sinks;
+    return launch_flash_prefill(c, f, st);
+}
+
 // q -> att, the head gates applied.  Few rows: the queries are taken into the latent space (q_lat[h] = W_uk[h]^T q[h]) and
 // attend the latent pages themselves.  Many rows of one sequence: keys and values are expanded once for the pass.
-static int attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, const LatentMixerSpec &m, const juno_kvpool *pool, int layer,
+static int latent_attention(juno_ctx *c, StackNet *net, const StackLayerWeights &L, const LatentMixerSpec &m, const juno_kvpool *pool, int layer,
                      const RowSet &rows, int n_splits, int len_bound, cudaStream_t st) {
     const int n = rows.n, dt = net->dt, H = m.heads, rp = m.rp(), dp = m.dp(), vp = m.vp();
     unsigned *err = c->gemv_scratch.qerr;
     const float *gate = net->u + m.gate_col();
     GemmArgs g;
     g.M = n;
-    if (dt == DT_BF16 && rows.one_seq && n > kAbsorbRows && flash_fits(m)) {
+    if (dt == DT_BF16 && rows.one_seq && n > kAbsorbRows && flash_fits(dp, vp)) {
         JUNO_TRY(ensure_device(&net->ctx_lat, &net->ctx_lat_bytes, (size_t)len_bound * rp * 2));
         JUNO_TRY(ensure_device(&net->ctx_kv, &net->ctx_kv_bytes, (size_t)len_bound * H * (dp + vp) * 2));
         JUNO_TRY(launch_latent_gather(c, pool, layer, rows.slots, len_bound, net->ctx_lat, st));
@@ -299,48 +406,92 @@ int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
         g.ldaux = wp;
         return launch_gemm_rows(c, dt, g, err, st);
     };
-    // x += norm(z) of the sublayer that ended, and the next sublayer's normed input
-    auto residual = [&](const void *z, float g_z, bool more, float g_next) {
+    // the residual takes the result z of the sublayer that ended, and gives the next one its normed input
+    struct Sublayer {
+        const StackLayerWeights *w = nullptr;
+        bool ff = false;
+    };
+    auto hand_over = [&](Sublayer done, Sublayer next) {
+        const bool more = next.w != nullptr;
+        if (s.streams) {
+            StreamStepArgs a;
+            a.x = net->x;
+            a.streams = s.streams;
+            a.ldx = wp;
+            a.width = s.width;
+            a.n = n;
+            a.eps = s.eps;
+            if (done.w) {
+                const HyperConnection &hc = done.ff ? done.w->hc2 : done.w->hc1;
+                a.z = net->z;
+                a.ldz = wp;
+                a.mix = hc.mix;
+                a.out = hc.out;
+            }
+            if (more) {
+                a.in = (next.ff ? next.w->hc2 : next.w->hc1).in;
+                a.w = next.ff ? next.w->norm2_w : next.w->norm1_w;
+                a.h = net->h;
+                a.ldh = wp;
+            }
+            return launch_stream_step(c, dt, a, st);
+        }
         ResidNormArgs a;
         a.x = net->x;
         a.ldx = wp;
         a.width = s.width;
         a.n = n;
-        a.z = z;
+        a.z = done.w ? net->z : nullptr;
         a.ldz = wp;
-        a.g_z = g_z;
-        a.g_next = g_next;
+        a.g_z = done.w ? (done.ff ? done.w->norm2b : done.w->norm1b) : 0.f;
+        a.g_next = more ? (next.ff ? next.w->norm2 : next.w->norm1) : 0.f;
         a.eps = s.eps;
         a.h = more ? net->h : nullptr;
         a.ldh = wp;
         a.row_scale = net->row_scale;
         return launch_resid_norm(c, dt, a, st);
     };
-    JUNO_TRY(launch_embed_norm(c, dt, net->embed.w, net->embed.cols, s.width, s.vocab, net->embed_norm, s.eps, rows, net->x, wp, st));
-    JUNO_TRY(residual(nullptr, 0.f, true, net->layers[s.weights(0)].norm1));
+    // the result of a sublayer; the gated residual multiplies it by its gate
+    auto result = [&](const void *a, const StackMat &w) {
+        return s.streams ? product(a, w.cols, w, net->z, wp, GE_OP) : product(a, w.cols, w, net->z, wp, GE_MUL, nullptr, net->gate);
+    };
+    auto weights = [&](int l) { return &net->layers[(size_t)s.weights(l)]; };
+    if (s.streams)
+        JUNO_TRY(launch_stream_embed(c, dt, net->embed.w, net->embed.cols, s.width, s.vocab, s.streams, rows, net->x, wp, st));
+    else
+        JUNO_TRY(launch_embed_norm(c, dt, net->embed.w, net->embed.cols, s.width, s.vocab, net->embed_norm, s.eps, rows, net->x, wp, st));
+    JUNO_TRY(hand_over({}, {weights(0), false}));
     for (int l = 0; l < n_layers; l++) {
-        const StackLayerWeights &L = net->layers[s.weights(l)];
-        const LatentMixerSpec &m = s.layers[l].mix;
-        const bool last = l + 1 == n_layers;
-        const float next_norm1 = last ? 0.f : net->layers[s.weights(l + 1)].norm1;
-        // mixer
-        JUNO_TRY(product(net->h, wp, L.rg1, net->gate, wp, GE_SIGMOID, L.rg1_b));
-        ConvArgs cv{net->x, wp, s.width, net->row_scale, L.conv, s.taps, pool, l, net->hc, wp};
-        JUNO_TRY(launch_conv(c, dt, cv, rows, st));
-        JUNO_TRY(product(net->hc, wp, L.down, net->u, net->ldu, GE_F32));
-        LatentNormArgs ln{net->u, net->ldu, m.q_rank, m.kv_col(), m.kv_rank, L.dq_norm, L.dkv_norm, s.eps, net->cq, m.qp(), pool, l};
-        JUNO_TRY(launch_latent_norm(c, dt, ln, rows, st));
-        JUNO_TRY(product(net->cq, m.qp(), L.uq, net->q, m.heads * m.dp(), GE_OP));
-        JUNO_TRY(attention(c, net, L, m, pool, l, rows, n_splits, len_bound, st));
-        JUNO_TRY(product(net->att, m.heads * m.vp(), L.o, net->z, wp, GE_MUL, nullptr, net->gate));
-        const bool mlp = s.layers[l].ff > 0;
-        JUNO_TRY(residual(net->z, L.norm1b, mlp || !last, mlp ? L.norm2 : next_norm1));
-        if (!mlp) continue;
-        // feed-forward
-        JUNO_TRY(product(net->h, wp, L.rg2, net->gate, wp, GE_SIGMOID, L.rg2_b));
-        JUNO_TRY(product(net->h, wp, L.up, net->act, L.mdown.cols, GE_RELU2));
-        JUNO_TRY(product(net->act, L.mdown.cols, L.mdown, net->z, wp, GE_MUL, nullptr, net->gate));
-        JUNO_TRY(residual(net->z, L.norm2b, !last, next_norm1));
+        const StackLayerWeights &L = *weights(l);
+        const StackLayerSpec &spec = s.layers[(size_t)l];
+        const Sublayer next = {l + 1 < n_layers ? weights(l + 1) : nullptr, false};
+        if (!s.streams) JUNO_TRY(product(net->h, wp, L.rg1, net->gate, wp, GE_SIGMOID, L.rg1_b));
+        if (spec.mixer == MIX_GROUPED) {
+            JUNO_TRY(product(net->h, wp, L.qkv, net->u, L.qkv.rows, GE_F32, L.qkv_b));
+            JUNO_TRY(grouped_attention(c, net, L, pool, l, rows, n_splits, len_bound, st));
+        } else {
+            const LatentMixerSpec &m = spec.mix;
+            ConvArgs cv{net->x, wp, s.width, net->row_scale, L.conv, s.taps, pool, l, net->hc, wp};
+            JUNO_TRY(launch_conv(c, dt, cv, rows, st));
+            JUNO_TRY(product(net->hc, wp, L.down, net->u, net->ldu, GE_F32));
+            LatentNormArgs ln{net->u, net->ldu, m.q_rank, m.kv_col(), m.kv_rank, L.dq_norm, L.dkv_norm, s.eps, net->cq, m.qp(), pool, l};
+            JUNO_TRY(launch_latent_norm(c, dt, ln, rows, st));
+            JUNO_TRY(product(net->cq, m.qp(), L.uq, net->q, m.heads * m.dp(), GE_OP));
+            JUNO_TRY(latent_attention(c, net, L, m, pool, l, rows, n_splits, len_bound, st));
+        }
+        JUNO_TRY(result(net->att, L.o));
+        if (spec.ff == 0) {
+            JUNO_TRY(hand_over({&L, false}, next));
+            continue;
+        }
+        JUNO_TRY(hand_over({&L, false}, {&L, true}));
+        if (!s.streams) JUNO_TRY(product(net->h, wp, L.rg2, net->gate, wp, GE_SIGMOID, L.rg2_b));
+        if (spec.ff_kind == FF_GEGLU)
+            JUNO_TRY(product(net->h, wp, L.gu, net->act, L.mdown.cols, GE_GEGLU));
+        else
+            JUNO_TRY(product(net->h, wp, L.up, net->act, L.mdown.cols, GE_RELU2));
+        JUNO_TRY(result(net->act, L.mdown));
+        JUNO_TRY(hand_over({&L, true}, next));
     }
     return JUNO_OK;
 }
@@ -348,7 +499,10 @@ int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
 int stack_enqueue_logits(juno_ctx *c, StackNet *net, const int32_t *row_idx, int n, float *logits, cudaStream_t st) {
     const StackSpec &s = net->spec;
     JUNO_REQUIRE(n >= 1 && n <= net->logit_cap, "logits of %d rows exceed the buffer (%d)", n, net->logit_cap);
-    JUNO_TRY(launch_gather_norm(c, net->dt, net->x, s.wp(), s.width, row_idx, n, net->final_norm, s.eps, net->fin, s.wp(), st));
+    if (s.streams)
+        JUNO_TRY(launch_stream_gather(c, net->dt, net->x, s.streams, s.wp(), s.width, row_idx, n, net->final_w, s.eps, net->fin, s.wp(), st));
+    else
+        JUNO_TRY(launch_gather_norm(c, net->dt, net->x, s.wp(), s.width, row_idx, n, net->final_norm, s.eps, net->fin, s.wp(), st));
     GemmArgs g;
     g.a = net->fin;
     g.lda = s.wp();

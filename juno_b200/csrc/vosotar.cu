@@ -2,61 +2,46 @@
 // norms before and after every sublayer, a short causal convolution on the mixer's input, and an element-wise sigmoid gate on
 // every sublayer's result.  This file knows the keys of its config.json and the names of its tensors; the mechanisms
 // themselves are the generic ones of stack.cuh.
-#include "json.hpp"
-#include "stack.cuh"
+#include "stack_loader.cuh"
 
 namespace juno {
 
-static int get_int(const Json *o, const char *key, const char *where, int lo, int hi, int *out) {
-    const Json *v = o ? o->find(key) : nullptr;
-    int64_t t = 0;
-    JUNO_REQUIRE(v && v->to_int(lo, hi, &t), "config: %s.%s must be a whole number in [%d, %d]", where, key, lo, hi);
-    *out = (int)t;
-    return JUNO_OK;
-}
-static int get_float(const Json *o, const char *key, const char *where, float *out) {
-    const Json *v = o ? o->find(key) : nullptr;
-    JUNO_REQUIRE(v && v->kind == Json::NUMBER, "config: %s.%s must be a number", where, key);
-    *out = (float)v->num;
-    return JUNO_OK;
-}
-
 int vosotar_spec(const Json &cfg, StackSpec *spec) {
     constexpr int kMax = 1 << 20;
-    JUNO_TRY(get_int(&cfg, "width", "model", 1, 49152, &spec->width));
-    JUNO_TRY(get_int(&cfg, "vocab", "model", 1, 1 << 24, &spec->vocab));
-    JUNO_TRY(get_float(cfg.find("norm"), "eps", "norm", &spec->eps));
-    JUNO_TRY(get_int(cfg.find("canon"), "taps", "canon", 1, 64, &spec->taps));
+    JUNO_TRY(cfg_int(&cfg, "width", "model", 1, 49152, &spec->width));
+    JUNO_TRY(cfg_int(&cfg, "vocab", "model", 1, 1 << 24, &spec->vocab));
+    JUNO_TRY(cfg_float(cfg.find("norm"), "eps", "norm", &spec->eps));
+    JUNO_TRY(cfg_int(cfg.find("canon"), "taps", "canon", 1, 64, &spec->taps));
     const Json *layers = cfg.find("layers");
     JUNO_REQUIRE(layers && layers->kind == Json::ARRAY && !layers->arr.empty(), "config: layers must be a non-empty list");
     for (size_t i = 0; i < layers->arr.size(); i++) {
         const Json &e = layers->arr[i];
         const std::string w = "layers[" + std::to_string(i) + "]";
         StackLayerSpec L;
-        const Json *type = e.find("type");
-        JUNO_REQUIRE(type && type->kind == Json::STRING, "config: %s.type is missing", w.c_str());
-        if (type->str != "latent_attention") {
-            set_error("config: %s: mixer '%s' is not part of this design", w.c_str(), type->str.c_str());
+        L.source = (int)i;
+        std::string type, kind;
+        JUNO_TRY(cfg_string(&e, "type", w.c_str(), &type));
+        if (type != "latent_attention") {
+            set_error("config: %s: mixer '%s' is not part of this design", w.c_str(), type.c_str());
             return JUNO_ERR_UNSUPPORTED;
         }
         const Json *m = e.find("mixer");
         const std::string wm = w + ".mixer";
-        JUNO_TRY(get_int(m, "heads", wm.c_str(), 1, 65535, &L.mix.heads));
-        JUNO_TRY(get_int(m, "dim", wm.c_str(), 1, kMax, &L.mix.dim));
-        JUNO_TRY(get_int(m, "vdim", wm.c_str(), 1, kMax, &L.mix.vdim));
-        JUNO_TRY(get_int(m, "q_rank", wm.c_str(), 1, kMax, &L.mix.q_rank));
-        JUNO_TRY(get_int(m, "kv_rank", wm.c_str(), 1, 2048, &L.mix.kv_rank));
-        JUNO_TRY(get_float(m, "scale", wm.c_str(), &L.mix.scale));
+        JUNO_TRY(cfg_int(m, "heads", wm.c_str(), 1, 65535, &L.mix.heads));
+        JUNO_TRY(cfg_int(m, "dim", wm.c_str(), 1, kMax, &L.mix.dim));
+        JUNO_TRY(cfg_int(m, "vdim", wm.c_str(), 1, kMax, &L.mix.vdim));
+        JUNO_TRY(cfg_int(m, "q_rank", wm.c_str(), 1, kMax, &L.mix.q_rank));
+        JUNO_TRY(cfg_int(m, "kv_rank", wm.c_str(), 1, 2048, &L.mix.kv_rank));
+        JUNO_TRY(cfg_float(m, "scale", wm.c_str(), &L.mix.scale));
         JUNO_REQUIRE(L.mix.scale > 0.f, "config: %s.scale must be positive", wm.c_str());
         const Json *mlp = e.find("mlp");
         if (mlp && !mlp->is_null()) {
-            const Json *kind = mlp->find("kind");
-            JUNO_REQUIRE(kind && kind->kind == Json::STRING, "config: %s.mlp.kind is missing", w.c_str());
-            if (kind->str != "dense") {
-                set_error("config: %s: feed-forward '%s' is not part of this design", w.c_str(), kind->str.c_str());
+            JUNO_TRY(cfg_string(mlp, "kind", (w + ".mlp").c_str(), &kind));
+            if (kind != "dense") {
+                set_error("config: %s: feed-forward '%s' is not part of this design", w.c_str(), kind.c_str());
                 return JUNO_ERR_UNSUPPORTED;
             }
-            JUNO_TRY(get_int(mlp, "ff", (w + ".mlp").c_str(), 1, kMax, &L.ff));
+            JUNO_TRY(cfg_int(mlp, "ff", (w + ".mlp").c_str(), 1, kMax, &L.ff));
         }
         const Json *src = e.find("weights_of");
         if (src && !src->is_null()) {
@@ -79,47 +64,7 @@ int vosotar_spec(const Json &cfg, StackSpec *spec) {
 }
 
 namespace {
-struct Loader {
-    juno_ctx *c;
-    const juno_safetensors *f;
-    StackNet *net;
-
-    // The tensor of that name with exactly that shape (a single number: one element, any rank).
-    int get(const std::string &name, std::vector<int64_t> shape, const StTensor **out) {
-        const StTensor *t = f->find(name);
-        JUNO_REQUIRE(t, "tensor %s is missing", name.c_str());
-        JUNO_REQUIRE(t->dtype == ST_BF16 || t->dtype == ST_F32, "tensor %s: weights must be BF16 or F32", name.c_str());
-        const bool ok = shape.empty() ? t->nelems == 1 : t->shape == shape;
-        if (!ok) {
-            std::string have, want;
-            for (int64_t d : t->shape) have += (have.empty() ? "" : "x") + std::to_string(d);
-            for (int64_t d : shape) want += (want.empty() ? "" : "x") + std::to_string(d);
-            set_error("tensor %s has shape [%s], expected [%s]", name.c_str(), have.c_str(), want.c_str());
-            return JUNO_ERR_INVALID_ARG;
-        }
-        *out = t;
-        return JUNO_OK;
-    }
-    int number(const std::string &name, float *out) {
-        const StTensor *t;
-        JUNO_TRY(get(name, {}, &t));
-        *out = st_value(f, *t, 0);
-        return JUNO_OK;
-    }
-    int vector(const std::string &name, int n, int padded, float **out) {
-        const StTensor *t;
-        JUNO_TRY(get(name, {n}, &t));
-        std::vector<float> v((size_t)padded, 0.f);
-        for (int i = 0; i < n; i++) v[(size_t)i] = st_value(f, *t, i);
-        return stack_upload_f32(c, net, v, out);
-    }
-    int matrix(const std::string &name, int rows, int cols, StackMat *out) {
-        const StTensor *t;
-        JUNO_TRY(get(name, {rows, cols}, &t));
-        HostMat m(net->dt, pad16(rows), pad16(cols));
-        m.put(f, *t, 0, 0, rows, cols, 0, 0);
-        return stack_upload(c, net, m, out);
-    }
+struct Loader : StackLoader {
     int mixer(const std::string &p, const LatentMixerSpec &s, StackLayerWeights *L) {
         const int W = net->spec.width, wp = net->spec.wp(), dt = net->dt, H = s.heads;
         const StTensor *dq, *dkv, *g, *uq, *uk, *uv, *o;
@@ -138,13 +83,11 @@ struct Loader {
         JUNO_TRY(get(p + "uv", {(int64_t)H * s.vdim, s.kv_rank}, &uv));
         JUNO_TRY(get(p + "o", {W, (int64_t)H * s.vdim}, &o));
         HostMat muq(dt, H * s.dp(), s.qp()), mukv(dt, H * (s.dp() + s.vp()), s.rp()), mukt(dt, H * s.rp(), s.dp()), mo(dt, wp, H * s.vp());
-        for (int h = 0; h < H; h++) {
-            muq.put(f, *uq, (int64_t)h * s.dim, 0, s.dim, s.q_rank, h * s.dp(), 0);
-            mukv.put(f, *uk, (int64_t)h * s.dim, 0, s.dim, s.kv_rank, h * s.dp(), 0);
-            mukv.put(f, *uv, (int64_t)h * s.vdim, 0, s.vdim, s.kv_rank, H * s.dp() + h * s.vp(), 0);
-            mukt.put_transposed(f, *uk, (int64_t)h * s.dim, 0, s.dim, s.kv_rank, h * s.rp(), 0);
-            mo.put(f, *o, 0, (int64_t)h * s.vdim, W, s.vdim, 0, h * s.vp());
-        }
+        put_heads(&muq, *uq, H, s.dim, s.dp(), s.q_rank, 0);
+        put_heads(&mukv, *uk, H, s.dim, s.dp(), s.kv_rank, 0);
+        put_heads(&mukv, *uv, H, s.vdim, s.vp(), s.kv_rank, H * s.dp());
+        put_head_columns(&mo, *o, H, s.vdim, s.vp(), W);
+        for (int h = 0; h < H; h++) mukt.put_transposed(f, *uk, (int64_t)h * s.dim, 0, s.dim, s.kv_rank, h * s.rp(), 0);
         JUNO_TRY(stack_upload(c, net, muq, &L->uq));
         JUNO_TRY(stack_upload(c, net, mukv, &L->ukv));
         JUNO_TRY(stack_upload(c, net, mukt, &L->ukt));
@@ -194,7 +137,7 @@ int vosotar_load(juno_ctx *c, const juno_safetensors *f, const StackSpec &spec, 
     StackNet *net = new StackNet();
     net->spec = spec;
     net->dt = dt;
-    Loader l{c, f, net};
+    Loader l{{c, f, net}};
     const int rc = l.all();
     if (rc != JUNO_OK) {
         stack_free(net);
