@@ -183,27 +183,94 @@ def vosotar_shapes(cfg: dict) -> dict:
     return t
 
 
+# ── Desilorn stacks ──────────────────────────────────────────────────────────────────────────────
+def desilorn_config(width: int, vocab: int, layers, streams: int = 2, loop=None, eps: float = 1e-6) -> dict:
+    """layers: dicts with heads, kv_heads, dim, vdim, scale, size (window or chunk), ff (0 or None: no feed-forward) and either
+    q_temp = (coef, every) (window attention) or rot = (base, dims) (chunk attention); loop: (start, stop, times)."""
+    out = []
+    for L in layers:
+        m = {k: L[k] for k in ("heads", "kv_heads", "dim", "vdim", "scale")}
+        m["mask"] = {"size": L["size"]}
+        if "rot" in L:
+            m["rot"] = {"base": L["rot"][0], "dims": L["rot"][1]}
+        else:
+            m["q_temp"] = {"coef": L["q_temp"][0], "every": L["q_temp"][1]}
+        out.append({"type": "attention_2" if "rot" in L else "attention", "mixer": m, "mlp": {"kind": "dense", "ff": L["ff"]} if L.get("ff") else None})
+    cfg = {"architecture": "Desilorn", "width": width, "vocab": vocab, "streams": streams, "norm": {"eps": eps}, "layers": out}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return cfg
+
+
+def desilorn_shapes(cfg: dict) -> dict:
+    """Tensor name -> (shape, fan-in or None) in file order."""
+    W, S = cfg["width"], cfg["streams"]
+    t = {"embed": ((cfg["vocab"], W), None), "final.norm": ((W,), None)}
+    for i, e in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", e["mixer"]
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        t[p + "norm1"] = ((W,), None)
+        for name, rows in (("q", H * d), ("k", G * d), ("v", G * dv)):
+            t.update({p + "mix." + name: ((rows, W), W), p + "mix." + name + ".b": ((rows,), None)})
+        if e["type"] == "attention_2":
+            t.update({p + "mix.q.norm": ((d,), None), p + "mix.k.norm": ((d,), None)})
+        else:
+            t[p + "mix.sink"] = ((H,), None)
+        t[p + "mix.o"] = ((W, H * dv), H * dv)
+        if e["mlp"] is not None:
+            ff = e["mlp"]["ff"]
+            t.update({p + "norm2": ((W,), None), p + "mlp.gate": ((ff, W), W), p + "mlp.up": ((ff, W), W), p + "mlp.down": ((W, ff), ff)})
+        for q in ("hc1.", "hc2.")[:1 if e["mlp"] is None else 2]:
+            t.update({p + q + "in": ((S,), None), p + q + "out": ((S,), None), p + q + "mix": ((S, S), None)})
+    return t
+
+
+def _desilorn_value(name: str, shape, rng) -> np.ndarray:
+    """Vectors and small matrices: mixtures near the identity, readings near the mean, norm weights near one."""
+    v = rng.standard_normal(shape)
+    if name.endswith("hc1.mix") or name.endswith("hc2.mix"):
+        return np.eye(shape[0]) + 0.15 * v
+    if name.endswith(".in"):
+        return 1.0 / shape[0] + 0.2 * v
+    if name.endswith(".out"):
+        return 0.7 + 0.3 * v
+    if name.endswith((".norm1", ".norm2")) or name == "final.norm":
+        return 0.3 * v  # stored as the distance from one
+    if name.endswith((".q.norm", ".k.norm")):
+        return 1.0 + 0.3 * v
+    return 0.3 * v if name.endswith(".b") else v
+
+
+def random_desilorn(cfg: dict, seed: int, fast: bool = False) -> dict:
+    """Random tensors (BF16 bit patterns) of a configuration, see random_stack."""
+    return random_stack(desilorn_shapes(cfg), seed, _desilorn_value, fast)
+
+
+# ── random tensors of a stack ────────────────────────────────────────────────────────────────────
+def _vosotar_value(name: str, shape, rng) -> np.ndarray:
+    v = rng.standard_normal(int(np.prod(shape)) if shape else 1)
+    return 0.5 * v if name.endswith(".b") else v if name == "embed" else 1.0 + 0.3 * v
+
+
 def random_vosotar(cfg: dict, seed: int, fast: bool = False) -> dict:
-    """Random tensors (BF16 bit patterns) of a configuration: fan-in scaled normals, norm weights round one, biases round zero.
+    """Random tensors (BF16 bit patterns) of a configuration: norm weights round one, biases round zero."""
+    return random_stack(vosotar_shapes(cfg), seed, _vosotar_value, fast)
+
+
+def random_stack(shapes: dict, seed: int, value, fast: bool = False) -> dict:
+    """Tensors (BF16 bit patterns) for name -> (shape, fan-in or None): fan-in scaled normals, else value(name, shape, rng).
     fast: large matrices repeat a drawn block (benchmarks, where only the shapes matter)."""
     from .safetensors_file import to_bf16
     rng = np.random.default_rng(seed)
     block = to_bf16(rng.standard_normal(1 << 20)) if fast else None
     out = {}
-    for name, (shape, fan) in vosotar_shapes(cfg).items():
+    for name, (shape, fan) in shapes.items():
         n = int(np.prod(shape)) if shape else 1
         if fast and n > (1 << 20):
             scale = int(round(np.log2(fan) / 2)) if fan else 0  # a power of two: an exponent shift of the block
             b = (block.astype(np.int32) - (scale << 7)).astype(np.uint16) if scale else block
             out[name] = np.resize(np.roll(b, int(rng.integers(1 << 20))), n).reshape(shape)
             continue
-        if fan:
-            v = rng.standard_normal(n) / np.sqrt(fan)
-        elif name.endswith(".b"):
-            v = 0.5 * rng.standard_normal(n)
-        elif name == "embed":
-            v = rng.standard_normal(n)
-        else:
-            v = 1.0 + 0.3 * rng.standard_normal(n)
+        v = rng.standard_normal(n) / np.sqrt(fan) if fan else value(name, shape, rng)
         out[name] = to_bf16(v).reshape(shape)
     return out

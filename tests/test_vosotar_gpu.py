@@ -7,15 +7,11 @@ import numpy as np
 import pytest
 
 from juno_b200 import synth
-from vosotarutil import CONFIGS, L, Pair, check, row_err
+from vosotarutil import CONFIGS, L, Pair, check, decode_all, row_err
 
 pytestmark = pytest.mark.gpu
 DTYPES = ["f32", "default"]
 NAMES = sorted(CONFIGS)
-
-
-def decode_all(h, rid, tokens, start=0):
-    return np.stack([h.forward_batch([rid], [[t]], [start + i])[0] for i, t in enumerate(tokens)])
 
 
 # ── whole prompts, decoding, portions ────────────────────────────────────────────────────────────
