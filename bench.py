@@ -213,7 +213,7 @@ def run_design(args):
     peaks = json.load(open(p)) if os.path.exists(p) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
     sampler = ClockSampler(0)
     sampler.start()
-    res = stackbench.run(args.sizes.split(","), [int(b) for b in args.batches.split(",")], args.ctx, args.steps, args.warmup,
+    res = stackbench.run(args.design, args.sizes.split(","), [int(b) for b in args.batches.split(",")], args.ctx, args.steps, args.warmup,
                          {k: float(peaks[k]) for k in ("hbm_gbs", "bf16_tflops")}, not args.no_llama)
     print(json.dumps({"design": args.design, "context": args.ctx, "steps": args.steps, "warmup": args.warmup, "data": "synthetic",
                       "dtype": "bf16", "clocks": sampler.result(), "sizes": res}), flush=True)
@@ -232,7 +232,7 @@ def main():
     ap.add_argument("--no-prefill", action="store_true", help="start decoding at an empty context (quick runs)")
     ap.add_argument("--chunked-prefill", action="store_true",
                     help="fill the prompt through juno_prefill (batched kernels, up to 64 positions per pass) instead of token by token")
-    ap.add_argument("--design", choices=["vosotar"], help="instead of the default workload: prefill and decode of a registered design "
+    ap.add_argument("--design", choices=["vosotar", "desilorn"], help="instead of the default workload: prefill and decode of a registered design "
                     "beside the LLaMA family at equal size (one GPU, one JSON line)")
     ap.add_argument("--sizes", default="small,medium,large", help="with --design")
     ap.add_argument("--batches", default="1,8,64", help="with --design: decode batches")

@@ -431,7 +431,13 @@ static int launch_inst(juno_ctx *c, const GvParams &p, size_t smem, cudaStream_t
             configured[c->device & 15] = true;
         }
     }
-    JUNO_CUDA_TRY(launch_pdl(gemv_rows_kernel<PRO, COLS>, dim3((unsigned)std::min(p.total_rt, c->sm_count)), dim3(kGvThreads), smem, st, p));
+    const dim3 grid((unsigned)std::min(p.total_rt, c->sm_count));
+    if (p.a.early) {
+        JUNO_CUDA_TRY(launch_pdl(gemv_rows_kernel<PRO, COLS>, grid, dim3(kGvThreads), smem, st, p));
+    } else {
+        gemv_rows_kernel<PRO, COLS><<<grid, kGvThreads, smem, st>>>(p);
+        JUNO_CUDA_TRY(cudaGetLastError());
+    }
     c->kernel_launches++;
     return JUNO_OK;
 }

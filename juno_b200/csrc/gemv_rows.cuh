@@ -36,6 +36,7 @@ struct GvArgs {
     int nseg = 0;
     GvSeg seg[3];
     int prologue = GVP_COPY;
+    bool early = true;  // may start while the kernel before it runs (programmatic dependent launch)
     // GVP_COPY: BF16 rows; group_rows > 0: rows group_rows * g .. of the matrix meet columns K * g .. of the operand
     const __nv_bfloat16 *in = nullptr;
     int ld_in = 0, in_cols = 0, group_rows = 0;

@@ -216,9 +216,7 @@ int stack_enqueue_step(juno_ctx *c, StackNet *net, const juno_kvpool *pool, cons
 void stack_step_done(const juno_ctx *c, StackNet *net, int n) {
     RowSet rows;
     rows.n = n;
-    net->last_x = 0;
-    if (!stack_fused_ok(c, net, rows)) return;
-    for (const StackLayerSpec &L : net->spec.layers) net->last_x ^= L.ff ? 0 : 1;  // one hand-over per sublayer
+    net->last_x = stack_fused_ok(c, net, rows) ? stack_decode_hand_overs(net, n) & 1 : 0;
 }
 
 int stack_residual(juno_ctx *c, StackNet *net, int n, const float **out, cudaStream_t st) {

@@ -157,6 +157,7 @@ int stack_enqueue_layers(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
 int stack_enqueue_logits(juno_ctx *c, StackNet *net, const int32_t *row_idx, int n, float *logits, cudaStream_t st);
 // The same for a decode step of few sequences, on fused products (stack_decode.cu).
 bool stack_fused_ok(const juno_ctx *c, const StackNet *net, const RowSet &rows);
+int stack_decode_hand_overs(const StackNet *net, int n);
 int stack_enqueue_decode(juno_ctx *c, StackNet *net, const juno_kvpool *pool, const RowSet &rows, int n_splits, cudaStream_t st);
 int stack_enqueue_decode_logits(juno_ctx *c, StackNet *net, int n, float *logits, cudaStream_t st);
 // One step of n sequences, logits included, on whichever of the two fits.

@@ -46,27 +46,66 @@ static GvSeg seg(const StackMat &w, int epi, void *out, int ldo) {
     return s;
 }
 
+// Up to this many sequences every CTA of a product reads the streams itself; from there on that costs more than a launch that
+// updates them and leaves the operand.
+constexpr int kStreamsInProduct = 2;
+static bool streams_in_product(const StackNet *net, int n) { return net->spec.streams > 0 && n <= kStreamsInProduct; }
+int stack_decode_hand_overs(const StackNet *net, int n) {  // times the newest residual rows change between x and x2
+    if (net->spec.streams && !streams_in_product(net, n)) return 0;
+    int k = 0;
+    for (const StackLayerSpec &L : net->spec.layers) k += L.ff ? 2 : 1;
+    return k;
+}
+
+static GvArgs from_rows(int n, const void *in, int ld, int cols, int K);
+
 // operand = norm of the residual, the pending sublayer result taken in first; what follows is a sublayer of `next`, or
 // (null) the output
-static GvArgs from_residual(StackNet *net, int n, const StackLayerWeights *next, bool ff) {
+static int from_residual(juno_ctx *c, StackNet *net, int n, const StackLayerWeights *next, bool ff, GvArgs *out, cudaStream_t st) {
+    const StackSpec &s = net->spec;
+    const int wp = s.wp();
     GvArgs a;
     a.n = n;
-    a.K = net->spec.wp();
-    a.width = net->spec.width;
-    a.eps = net->spec.eps;
-    if (net->spec.streams) {
+    a.K = wp;
+    a.width = s.width;
+    a.eps = s.eps;
+    a.x = net->last_x ? net->x2 : net->x;
+    if (s.streams) {
+        const float *in = next ? (ff ? next->hc2 : next->hc1).in : net->ones, *w = next ? (ff ? next->norm2_w : next->norm1_w) : net->final_w;
+        if (!streams_in_product(net, n)) {
+            StreamStepArgs t;
+            t.x = net->x;
+            t.streams = s.streams;
+            t.ldx = wp;
+            t.width = s.width;
+            t.n = n;
+            if (net->pending) {
+                t.z = net->z;
+                t.ldz = wp;
+                t.mix = net->pending_hc->mix;
+                t.out = net->pending_hc->out;
+                net->pending = false;
+            }
+            t.in = in;
+            t.w = w;
+            t.eps = s.eps;
+            t.h = net->h;
+            t.ldh = wp;
+            JUNO_TRY(launch_stream_step(c, net->dt, t, st));
+            *out = from_rows(n, net->h, wp, wp, wp);
+            return JUNO_OK;
+        }
         a.prologue = GVP_STREAMS;
-        a.streams = net->spec.streams;
-        a.hc_in = next ? (ff ? next->hc2 : next->hc1).in : net->ones;
-        a.norm_w = next ? (ff ? next->norm2_w : next->norm1_w) : net->final_w;
+        a.streams = s.streams;
+        a.hc_in = in;
+        a.norm_w = w;
     } else {
         a.prologue = GVP_RESIDUAL;
         a.g_next = next ? (ff ? next->norm2 : next->norm1) : net->final_norm;
     }
-    a.x = net->last_x ? net->x2 : net->x;
     if (net->pending) {
         a.z = net->dec_z;
-        if (net->spec.streams) {
+        if (s.streams) {
             a.hc_mix = net->pending_hc->mix;
             a.hc_out = net->pending_hc->out;
         } else {
@@ -76,7 +115,8 @@ static GvArgs from_residual(StackNet *net, int n, const StackLayerWeights *next,
         a.x_store = net->last_x ? net->x2 : net->x;
         net->pending = false;
     }
-    return a;
+    *out = a;
+    return JUNO_OK;
 }
 static GvArgs from_rows(int n, const void *in, int ld, int cols, int K) {
     GvArgs a;
@@ -95,7 +135,8 @@ static int latent_mixer(juno_ctx *c, StackNet *net, const juno_kvpool *pool, int
     const LatentMixerSpec &m = s.layers[l].mix;
     const int n = rows.n, wp = s.wp(), H = m.heads, rp = m.rp(), dp = m.dp(), vp = m.vp();
     {
-        GvArgs a = from_residual(net, n, &L, false);
+        GvArgs a;
+        JUNO_TRY(from_residual(c, net, n, &L, false, &a, st));
         a.conv_w = static_cast<const bf16 *>(L.conv);
         a.taps = s.taps;
         if (pool->state) {
@@ -155,7 +196,8 @@ static int latent_mixer(juno_ctx *c, StackNet *net, const juno_kvpool *pool, int
 static int grouped_mixer(juno_ctx *c, StackNet *net, const juno_kvpool *pool, int l, const RowSet &rows, int n_splits, cudaStream_t st) {
     const StackSpec &s = net->spec;
     const StackLayerWeights &L = net->layers[s.weights(l)];
-    GvArgs a = from_residual(net, rows.n, &L, false);
+    GvArgs a;
+    JUNO_TRY(from_residual(c, net, rows.n, &L, false, &a, st));
     a.nseg = 1;
     a.seg[0] = seg(L.qkv, GVE_F32, net->u, L.qkv.rows);
     a.seg[0].bias = L.qkv_b;
@@ -174,10 +216,14 @@ int stack_enqueue_decode(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
     else
         JUNO_TRY(launch_embed_norm(c, net->dt, net->embed.w, net->embed.cols, s.width, s.vocab, net->embed_norm, s.eps, rows, net->x, wp, st));
     // the result of a sublayer stays pending: the next product takes it into the residual
-    auto sublayer_out = [&](const void *in, const StackMat &w, float g, const HyperConnection &hc) {
+    auto sublayer_out = [&](const void *in, const StackMat &w, float g, const HyperConnection &hc, bool early) {
         GvArgs a = from_rows(n, in, w.cols, w.cols, w.cols);
+        a.early = early;
         a.nseg = 1;
-        a.seg[0] = seg(w, s.streams ? GVE_F32 : GVE_MUL, net->dec_z, wp);
+        if (s.streams && !streams_in_product(net, n))
+            a.seg[0] = seg(w, GVE_OP, net->z, wp);
+        else
+            a.seg[0] = seg(w, s.streams ? GVE_F32 : GVE_MUL, net->dec_z, wp);
         a.seg[0].aux = net->dec_gate;
         a.seg[0].ldaux = wp;
         net->pending = true;
@@ -189,22 +235,26 @@ int stack_enqueue_decode(juno_ctx *c, StackNet *net, const juno_kvpool *pool, co
         const StackLayerWeights &L = net->layers[s.weights(l)];
         const StackLayerSpec &spec = s.layers[l];
         JUNO_TRY(spec.mixer == MIX_GROUPED ? grouped_mixer(c, net, pool, l, rows, n_splits, st) : latent_mixer(c, net, pool, l, rows, n_splits, st));
-        JUNO_TRY(sublayer_out(net->att, L.o, L.norm1b, L.hc1));
+        // started early, W_o's CTAs (each wants a whole SM) would wait among the small ones of the grouped attention, and the
+        // product after it then ran at half its rate
+        JUNO_TRY(sublayer_out(net->att, L.o, L.norm1b, L.hc1, spec.mixer != MIX_GROUPED));
         if (spec.ff == 0) continue;
-        GvArgs a = from_residual(net, n, &L, true);
+        GvArgs a;
+        JUNO_TRY(from_residual(c, net, n, &L, true, &a, st));
         if (!s.streams) {
             a.seg[a.nseg] = seg(L.rg2, GVE_SIGMOID, net->dec_gate, wp);
             a.seg[a.nseg++].bias = L.rg2_b;
         }
         a.seg[a.nseg++] = spec.ff_kind == FF_GEGLU ? seg(L.gu, GVE_GEGLU, net->act, L.mdown.cols) : seg(L.up, GVE_RELU2, net->act, L.mdown.cols);
         JUNO_TRY(launch_gemv_rows(c, a, st));
-        JUNO_TRY(sublayer_out(net->act, L.mdown, L.norm2b, L.hc2));
+        JUNO_TRY(sublayer_out(net->act, L.mdown, L.norm2b, L.hc2, true));
     }
     return JUNO_OK;
 }
 
 int stack_enqueue_decode_logits(juno_ctx *c, StackNet *net, int n, float *logits, cudaStream_t st) {
-    GvArgs a = from_residual(net, n, nullptr, false);
+    GvArgs a;
+    JUNO_TRY(from_residual(c, net, n, nullptr, false, &a, st));
     a.nseg = 1;
     a.seg[0] = seg(net->head, GVE_F32, logits, net->spec.vocab);
     a.seg[0].n_store = net->spec.vocab;

@@ -1,6 +1,6 @@
 """Prefill and decode throughput of a registered design (random weights) beside the framework's LLaMA family at equal size.
 
-    python bench.py --design vosotar [--sizes small,medium,large] [--steps K] [--warmup W]
+    python bench.py --design vosotar|desilorn [--sizes small,medium,large] [--steps K] [--warmup W]
 
 Equal size: the same width, feed-forward width, layers, vocabulary and number of query heads; the LLaMA model is Q4_K_M, as the
 framework serves it.  Timed with CUDA events on the context's stream after warm-up; the weights of a step exceed L2.
@@ -18,7 +18,7 @@ from .handler import B200TransformerHandler
 from .matvec import GpuContext
 from .safetensors_file import write_model_folder
 
-# width, heads, feed-forward, q_rank, kv_rank, layers (dim = vdim = 128)
+# width, heads, feed-forward, q_rank, kv_rank, layers (heads of 128; grouped attention has 8 key/value heads, as LLaMA)
 SIZES = {"small": (2048, 16, 8192, 768, 512, 8), "medium": (4096, 32, 14336, 1536, 512, 4), "large": (8192, 64, 28672, 1536, 512, 2)}
 VOCAB = 32000
 
@@ -29,14 +29,26 @@ def vosotar_model(size: str) -> dict:
     return synth.vosotar_config(w, VOCAB, [dict(one) for _ in range(n)])
 
 
+def desilorn_model(size: str) -> dict:
+    """Window and chunk layers in turn, spans longer than the measured contexts (every cached key is read, as in LLaMA)."""
+    w, heads, ff, _, _, n = SIZES[size]
+    one = dict(heads=heads, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, ff=ff)
+    kinds = (dict(one, size=8192, rot=(500000.0, 128)), dict(one, size=4096, q_temp=(0.1, 1024)))
+    return synth.desilorn_config(w, VOCAB, [dict(kinds[i % 2]) for i in range(n)], streams=4)
+
+
+DESIGNS = {"vosotar": (vosotar_model, synth.vosotar_shapes, synth.random_vosotar),
+           "desilorn": (desilorn_model, synth.desilorn_shapes, synth.random_desilorn)}
+
+
 def llama_arch(size: str) -> synth.Arch:
     w, heads, ff, _, _, n = SIZES[size]
     return synth.Arch(w, n, heads, 8, ff, VOCAB, 1e-5, 500000.0)
 
 
-def matrix_params(cfg: dict) -> float:
-    """Weights every position of a prompt meets, layers only."""
-    return float(sum(np.prod(s) for n, (s, _) in synth.vosotar_shapes(cfg).items() if n.startswith("l") and len(s) == 2 and "canon" not in n))
+def matrix_params(shapes: dict) -> float:
+    """Weights every position of a prompt meets in matrix products, layers only."""
+    return float(sum(np.prod(s) for n, (s, fan) in shapes.items() if n.startswith("l") and len(s) == 2 and fan and "canon" not in n))
 
 
 def _events():
@@ -106,16 +118,17 @@ def measure(h, ctx, batches, context: int, warmup: int, steps: int, prefill_step
     return out
 
 
-def run(sizes, batches, context: int, steps: int, warmup: int, peaks: dict, llama: bool = True) -> dict:
+def run(design: str, sizes, batches, context: int, steps: int, warmup: int, peaks: dict, llama: bool = True) -> dict:
+    model, shapes, random_model = DESIGNS[design]
     ctx = GpuContext.shared(0)
     res = {}
     hbm, tf = peaks["hbm_gbs"], peaks["bf16_tflops"]
     room = context + 2 * steps + warmup + 16
     for size in sizes:
-        cfg = vosotar_model(size)
+        cfg = model(size)
         d = tempfile.mkdtemp(prefix="stackbench")
         try:
-            write_model_folder(d, cfg, synth.random_vosotar(cfg, 7, fast=True))
+            write_model_folder(d, cfg, random_model(cfg, 7, fast=True))
             h = B200TransformerHandler.open(d, ctx, max_batch=max(batches), max_seqs=max(batches) + 1, max_ctx=room)
         finally:
             shutil.rmtree(d, ignore_errors=True)
@@ -123,7 +136,7 @@ def run(sizes, batches, context: int, steps: int, warmup: int, peaks: dict, llam
         m = cfg["layers"][0]["mixer"]
         n_layers, H = len(cfg["layers"]), m["heads"]
         attn = 2.0 * context * context / 2 * H * (m["dim"] + m["vdim"]) * n_layers
-        flops = 2.0 * context * matrix_params(cfg) + attn
+        flops = 2.0 * context * matrix_params(shapes(cfg)) + attn
         r["prefill"]["tflops"] = flops / r["prefill"]["ms"] / 1e9
         r["prefill"]["of_measured"] = r["prefill"]["tflops"] / tf
         r["prefill"]["attention_tflops"] = attn / r["prefill"]["profile"]["attention"]["ms"] / 1e9
@@ -131,8 +144,9 @@ def run(sizes, batches, context: int, steps: int, warmup: int, peaks: dict, llam
             nbytes = h.arch.weight_bytes + int(b) * (context + 1.5 * steps + warmup) * h.arch.cache_bytes_per_token
             v["gbs"] = nbytes / v["ms_per_step"] / 1e6
             v["of_measured"] = v["gbs"] / hbm
+            v["attention_gbs"] = int(b) * (context + 2 * steps + warmup) * h.arch.cache_bytes_per_token / v["profile"]["attention"]["ms"] / 1e6
         h.release_gpu_resources()
-        res[size] = {"vosotar": r}
+        res[size] = {design: r}
         if not llama:
             continue
         arch = llama_arch(size)
@@ -151,6 +165,7 @@ def run(sizes, batches, context: int, steps: int, warmup: int, peaks: dict, llam
             nbytes = wb + int(b) * (context + 1.5 * steps + warmup) * 4.0 * arch.kv_dim * arch.n_layers
             v["gbs"] = nbytes / v["ms_per_step"] / 1e6
             v["of_measured"] = v["gbs"] / hbm
+            v["attention_gbs"] = int(b) * (context + 2 * steps + warmup) * 4.0 * arch.kv_dim * arch.n_layers / v["profile"]["attention"]["ms"] / 1e6
         h.release_gpu_resources()
         res[size]["llama_q4_k_m"] = r
     return res
