@@ -264,8 +264,10 @@ int juno_model_load_gguf(juno_model *m, juno_gguf *g);
  * Opens a model by what the path holds and returns it finalized, ready for juno_model_seq_create and the step calls:
  *   - a folder with config.json and model.safetensors: the design that config.json's "architecture" names.  Registered:
  *     "Vosotar" (latent attention without positions over latent pages, squared-ReLU feed-forwards, scalar norms, a short
- *     convolution on the mixer's input whose state belongs to the sequence, sigmoid-gated residuals).  An architecture
- *     that is not registered gives JUNO_ERR_UNSUPPORTED;
+ *     convolution on the mixer's input whose state belongs to the sequence, sigmoid-gated residuals) and "Desilorn" (grouped
+ *     attention over windows with a distance bias and over chunks with a rotation, softmax sinks, gated GELU feed-forwards,
+ *     hyper-connected residual streams, a span of layers that runs several times).  An architecture that is not registered
+ *     gives JUNO_ERR_UNSUPPORTED;
  *   - a file: GGUF, the quantised LLaMA family (juno_gguf_model_cfg, juno_model_load_gguf).
  * Sequences of a model with a convolution state can be continued at their end, restarted at 0, or rewound by the few
  * positions the state reaches back; anything else is JUNO_ERR_INVALID_ARG.  One GPU. */

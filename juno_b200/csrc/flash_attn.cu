@@ -20,13 +20,13 @@ struct FlashParams {
     int max_pages, row_width;
 };
 // D: most dimensions per head; MT: 16-row tiles per warp; PAGED: keys and values from the sequence's pages, with key spans,
-// distance slopes and sinks (scores are kept in the log2 domain then)
-template <int D, int MT, bool PAGED>
+// distance slopes and sinks (scores are kept in the log2 domain then); EXACT: query, key and value size are D
+template <int D, int MT, bool PAGED, bool EXACT>
 __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_kernel(const FlashParams p) {
     extern __shared__ __align__(16) uint8_t sm[];
     constexpr int BR = 64 * MT, NK = D / 16, NV = D / 16;
     const FlashArgs &a = p.a;
-    const int dp = a.dim, vp = a.vdim, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
+    const int dp = EXACT ? D : a.dim, vp = EXACT ? D : a.vdim, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
     bf16 *qs = reinterpret_cast<bf16 *>(sm);
     bf16 *ks = qs + BR * kp;                 // [2][64][kp]
     bf16 *vs = ks + 2 * kFlKeys * kp;        // [2][64][vpitch]
@@ -61,6 +61,25 @@ __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_ke
     };
     auto load_kv = [&](int j, int buf) {
         const bf16 *base = PAGED ? p.plane : kv;
+        if (EXACT && j >= first && j + kFlKeys <= len) {  // every row exists: a thread's pieces lie in one column of them
+            constexpr int RS = kFlThreads / (D / 8);  // rows between them
+            const bf16 *ksrc = base + kvh * dp + kch0 * 8, *vsrc = base + G * dp + kvh * vp + kch0 * 8;
+            const uint32_t kd = smem_addr(ks + ((size_t)buf * kFlKeys + kr0) * kp + kch0 * 8), vd = smem_addr(vs + ((size_t)buf * kFlKeys + kr0) * vpitch + kch0 * 8);
+            const size_t step = PAGED ? (size_t)p.row_width : (size_t)a.ldkv;
+#pragma unroll
+            for (int pg = 0; pg < kFlKeys / kPageTokens; pg++) {
+                const size_t row0 = PAGED ? (size_t)table[(j >> 4) + pg] * kPageTokens : (size_t)j + pg * kPageTokens;
+                size_t off = (row0 + kr0) * step;
+#pragma unroll
+                for (int r = 0; r < kPageTokens; r += RS, off += RS * step) {
+                    const uint32_t d = (uint32_t)((pg * kPageTokens + r) * kp) * 2;  // kp == vpitch
+                    cp16(kd + d, ksrc + off, true);
+                    cp16(vd + d, vsrc + off, true);
+                }
+            }
+            cp_commit();
+            return;
+        }
         load_rows(base + kvh * dp, smem_addr(ks + (size_t)buf * kFlKeys * kp), kp, j, kr0, kch0, krs, kcs, kc);
         load_rows(base + G * dp + kvh * vp, smem_addr(vs + (size_t)buf * kFlKeys * vpitch), vpitch, j, vr0, vch0, vrs, vcs, vc);
         cp_commit();
@@ -133,14 +152,17 @@ __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_ke
             for (int e2 = 0; e2 < 2; e2++) {  // rows g and g + 8
                 const int pos = a.pos0 + r0 + wrow + m * 16 + g + e2 * 8;
                 float mv = mx[m][e2];
-                if (PAGED) {
+                if (PAGED && a.slopes) {
+                    const float b0 = (float)(j + 2 * t - pos) * slope;
 #pragma unroll
                     for (int i = 0; i < kFlKeys / 8; i++)
 #pragma unroll
-                        for (int e = 0; e < 2; e++) {
-                            float &v = s[m][i][e2 * 2 + e];
-                            v = fmaf((float)(j + i * 8 + 2 * t + e - pos), slope, v * p.scale_log2);
-                        }
+                        for (int e = 0; e < 2; e++) s[m][i][e2 * 2 + e] = fmaf(s[m][i][e2 * 2 + e], p.scale_log2, fmaf((float)(i * 8 + e), slope, b0));
+                } else if (PAGED) {
+#pragma unroll
+                    for (int i = 0; i < kFlKeys / 8; i++)
+#pragma unroll
+                        for (int e = 0; e < 2; e++) s[m][i][e2 * 2 + e] *= p.scale_log2;
                 }
                 if (j + kFlKeys - 1 > pos || (PAGED && j < lo[m][e2])) {
 #pragma unroll
@@ -222,8 +244,8 @@ __global__ void __launch_bounds__(kFlThreads, D <= 128 ? 2 : 1) flash_prefill_ke
 }
 
 // ───────────────────────────── launches ───────────────────────────────────────────────────
-template <int D, int MT, bool PAGED>
-static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
+template <int D, int MT, bool PAGED, bool EXACT>
+static int flash_inst(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
     constexpr int BR = 64 * MT;
     const size_t smem = ((size_t)(BR + 2 * kFlKeys) * (p.a.dim + 8) + (size_t)2 * kFlKeys * (p.a.vdim + 8)) * 2;
     static std::mutex mu;
@@ -231,14 +253,19 @@ static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
     {
         std::lock_guard<std::mutex> lk(mu);
         if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(flash_prefill_kernel<D, MT, PAGED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(flash_prefill_kernel<D, MT, PAGED, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             have[c->device & 15] = smem;
         }
     }
-    flash_prefill_kernel<D, MT, PAGED><<<dim3((unsigned)p.a.heads, (unsigned)((p.a.n + BR - 1) / BR)), kFlThreads, smem, st>>>(p);
+    flash_prefill_kernel<D, MT, PAGED, EXACT><<<dim3((unsigned)p.a.heads, (unsigned)((p.a.n + BR - 1) / BR)), kFlThreads, smem, st>>>(p);
     JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;
+}
+
+template <int D, int MT, bool PAGED>
+static int flash_launch(juno_ctx *c, const FlashParams &p, cudaStream_t st) {
+    return p.a.dim == D && p.a.vdim == D ? flash_inst<D, MT, PAGED, true>(c, p, st) : flash_inst<D, MT, PAGED, false>(c, p, st);
 }
 
 int launch_flash_prefill(juno_ctx *c, const FlashArgs &a, cudaStream_t st) {

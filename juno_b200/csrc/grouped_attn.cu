@@ -166,12 +166,13 @@ static size_t grouped_split_smem(int dp, int vp) {
     return (size_t)16 * (dp + 8) * 2 + std::max(ring, merge);
 }
 
-// ND: 16-column steps of a head at most; FUSED: queries, keys and values from the projections
-template <int ND, bool FUSED>
+// ND: 16-column steps of a head at most; FUSED: queries, keys and values from the projections; DIM: query, key and value size
+// of a head when they are equal and a common number (every offset and bound folds), else 0
+template <int ND, bool FUSED, int DIM>
 __global__ void __launch_bounds__(kGdThreads) grouped_split_kernel(const __grid_constant__ GroupedSplitParams p) {
     extern __shared__ __align__(16) uint8_t sm[];
     const GroupedAttnArgs &a = p.g.a;
-    const int dp = a.dp, vp = a.vp, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
+    const int dp = DIM ? DIM : a.dp, vp = DIM ? DIM : a.vp, kp = dp + 8, vpitch = vp + 8, nk = dp >> 4, nv = vp >> 4;
     bf16 *qs = reinterpret_cast<bf16 *>(sm);  // [16][kp]
     uint8_t *pool_s = sm + 16 * kp * 2;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -191,6 +192,16 @@ __global__ void __launch_bounds__(kGdThreads) grouped_split_kernel(const __grid_
     const int kr0 = lane / kc, kch0 = lane - kr0 * kc, krs = 32 / kc, kcs = 32 - krs * kc;
     const int vr0 = lane / vc, vch0 = lane - vr0 * vc, vrs = 32 / vc, vcs = 32 - vrs * vc;
     auto load_part = [&](const bf16 *src, uint32_t dst, int pitch, int key0, int r, int ch, int rs, int chs, int nch) {
+        if (DIM && key0 >= lo && key0 + 15 <= pos) {  // every row is seen: a lane's pieces lie in one column of them
+            src += (size_t)r * p.g.row_width + ch * 8;
+            dst += (uint32_t)(r * pitch + ch * 8) * 2;
+#pragma unroll
+            for (int i = 0; i < 16; i += 32 / (DIM ? DIM / 8 : 1)) {
+                cp16(dst + (uint32_t)(i * pitch) * 2, src, true);
+                src += (size_t)rs * p.g.row_width;
+            }
+            return;
+        }
         while (r < 16) {
             const bool ok = key0 + r >= lo && key0 + r <= pos;
             cp16(dst + (uint32_t)(r * pitch + ch * 8) * 2, ok ? src + (size_t)r * p.g.row_width + ch * 8 : plane, ok);
@@ -284,16 +295,20 @@ __global__ void __launch_bounds__(kGdThreads) grouped_split_kernel(const __grid_
                 mma16816(s[1], qa[k], b[2], b[3]);
             }
         float f[2];
+        const bool whole = ti * 16 >= lo && ti * 16 + 15 <= pos;
 #pragma unroll
         for (int e2 = 0; e2 < 2; e2++) {
             float m = mx[e2];
+            const float slope = e2 ? slope1 : slope0;
 #pragma unroll
             for (int i = 0; i < 2; i++)
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     const int key = ti * 16 + i * 8 + 2 * t + e;
                     float &v = s[i][e2 * 2 + e];
-                    v = key >= lo && key <= pos ? fmaf((float)(key - pos), e2 ? slope1 : slope0, v * scale_l2) : -INFINITY;
+                    v *= scale_l2;
+                    if (a.slopes) v = fmaf((float)(key - pos), slope, v);
+                    if (!whole && (key < lo || key > pos)) v = -INFINITY;
                     m = fmaxf(m, v);
                 }
             m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
@@ -312,11 +327,9 @@ __global__ void __launch_bounds__(kGdThreads) grouped_split_kernel(const __grid_
             ls[e2] = ls[e2] * f[e2] + sum;
         }
         const uint32_t pa[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
+        if (__any_sync(0xffffffffu, f[0] != 1.f || f[1] != 1.f)) {  // a maximum has moved
 #pragma unroll
-        for (int i = 0; i < ND; i++)
-            if (i < nv) {
-                uint32_t b[4];
-                ldsm4_trans(b, smem_addr(vs + lr * vpitch + i * 16 + lc));
+            for (int i = 0; i < ND; i++)
 #pragma unroll
                 for (int k = 0; k < 2; k++) {
                     o[i][k][0] *= f[0];
@@ -324,6 +337,12 @@ __global__ void __launch_bounds__(kGdThreads) grouped_split_kernel(const __grid_
                     o[i][k][2] *= f[1];
                     o[i][k][3] *= f[1];
                 }
+        }
+#pragma unroll
+        for (int i = 0; i < ND; i++)
+            if (i < nv) {
+                uint32_t b[4];
+                ldsm4_trans(b, smem_addr(vs + lr * vpitch + i * 16 + lc));
                 mma16816(o[i][0], pa, b[0], b[1]);
                 mma16816(o[i][1], pa, b[2], b[3]);
             }
@@ -518,21 +537,21 @@ int grouped_pick_splits(const juno_ctx *c, int n, int heads, int kv_heads, int d
 size_t grouped_part_floats(const juno_ctx *c, int vp) { return (size_t)4 * c->sm_count * 16 * (vp + 2); }
 size_t grouped_counters(const juno_ctx *c) { return (size_t)4 * c->sm_count; }
 
-template <int ND, bool FUSED>
+template <int ND, bool FUSED, int DIM = 0>
 static int split_launch(juno_ctx *c, const GroupedSplitParams &p, dim3 grid, size_t smem, cudaStream_t st) {
     static std::mutex mu;
     static size_t have[16] = {0};
     {
         std::lock_guard<std::mutex> lk(mu);
         if (smem > have[c->device & 15]) {
-            JUNO_CUDA_TRY(cudaFuncSetAttribute(grouped_split_kernel<ND, FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            JUNO_CUDA_TRY(cudaFuncSetAttribute(grouped_split_kernel<ND, FUSED, DIM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             have[c->device & 15] = smem;
         }
     }
     if (FUSED)
-        JUNO_CUDA_TRY(launch_pdl(grouped_split_kernel<ND, FUSED>, grid, dim3(kGdThreads), smem, st, p));
+        JUNO_CUDA_TRY(launch_pdl(grouped_split_kernel<ND, FUSED, DIM>, grid, dim3(kGdThreads), smem, st, p));
     else
-        grouped_split_kernel<ND, FUSED><<<grid, kGdThreads, smem, st>>>(p);
+        grouped_split_kernel<ND, FUSED, DIM><<<grid, kGdThreads, smem, st>>>(p);
     JUNO_CUDA_TRY(cudaGetLastError());
     c->kernel_launches++;
     return JUNO_OK;
@@ -557,6 +576,8 @@ int launch_grouped_split(juno_ctx *c, const GroupedAttnArgs &a, int n_splits, bo
     const dim3 grid((unsigned)n_splits, (unsigned)(a.kv_heads * p.head_tiles), (unsigned)n);
     const size_t smem = grouped_split_smem(a.dp, a.vp);
     ProfScope prof(c, st, PROF_ATTN, 0);
+    if (a.dp == 64 && a.vp == 64) return fused ? split_launch<4, true, 64>(c, p, grid, smem, st) : split_launch<4, false, 64>(c, p, grid, smem, st);
+    if (a.dp == 128 && a.vp == 128) return fused ? split_launch<8, true, 128>(c, p, grid, smem, st) : split_launch<8, false, 128>(c, p, grid, smem, st);
     if (fused) {
         if (d <= 64) return split_launch<4, true>(c, p, grid, smem, st);
         if (d <= 128) return split_launch<8, true>(c, p, grid, smem, st);

@@ -29,6 +29,8 @@ CONFIGS = {
     "wide": synth.desilorn_config(96, 130, [C(3, 1, 200, 144, 90, 40, (50000.0, 120)), W(2, 1, 144, 256, 64, 56)], streams=5, loop=(0, 2, 3)),
     # heads wider than the tensor-core kernels take: the general kernel
     "bighead": synth.desilorn_config(64, 90, [W(2, 1, 272, 300, 40, 50), C(2, 2, 280, 16, 48, 0, (100.0, 280))], streams=2),
+    # heads of two hundred and fifty-six
+    "d256": synth.desilorn_config(80, 110, [W(3, 1, 256, 256, 130, 64), C(2, 2, 256, 256, 210, 0, (1e4, 64))], streams=3),
     # head sizes of real models
     "real": synth.desilorn_config(256, 300, [C(8, 2, 128, 128, 256, 256, (500000.0, 64)), W(8, 2, 128, 128, 128, 256, (0.1, 32))], streams=4, loop=(1, 2, 2)),
 }

@@ -36,7 +36,7 @@ def test_prompt_and_decoding_match_the_oracle(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["odd", "groups", "long", "wide", "real"])
+@pytest.mark.parametrize("name", ["odd", "groups", "long", "wide", "d256", "real"])
 def test_portions_of_any_size(tmp_path, name, dtype):
     p = Pair(tmp_path, CONFIGS[name], seed=2)
     toks = p.tokens(400, 1)
